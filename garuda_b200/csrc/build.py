@@ -42,6 +42,8 @@ KERNEL_LIBS: Dict[str, List[str]] = {
     # a norm after the sum, a gated recurrence per channel, a short convolution in front of attention:
     # built when a model first uses them
     "garuda_seq": ["post_norm.cu", "mingru.cu", "conv_qkv.cu"],
+    # a state space with one decay per head and token: built when a model first needs it
+    "garuda_ssd": ["state_space.cu"],
 }
 HOST_SOURCES = ["cache_manager.cpp", "scheduler.cpp", "step_batch.cpp", "bindings.cpp"]
 
@@ -157,7 +159,16 @@ def capped_attention_lib_name(key_dim: int, value_dim: int) -> str:
     return f"garuda_cattn_k{int(key_dim)}_v{int(value_dim)}"
 
 
+def ssd_lib_name(state_dim: int, head_dim: int) -> str:
+    """The state-space recurrence on the tensor cores is compiled per (state width, head width), when a
+    model first needs it."""
+    return f"garuda_ssdc_n{int(state_dim)}_p{int(head_dim)}"
+
+
 def _lib_recipe(name: str):
+    if name.startswith("garuda_ssdc_n"):
+        n, p = name[len("garuda_ssdc_n"):].split("_p")
+        return ["ssd_chunk_mma.cu"], [f"-DGB_STATE_DIM={int(n)}", f"-DGB_HEAD_DIM={int(p)}"]
     if name.startswith("garuda_cattn_k"):
         kd, vd = name[len("garuda_cattn_k"):].split("_v")
         return ["attention_capped_mma.cu"], [f"-DGB_KEY_DIM={int(kd)}", f"-DGB_VALUE_DIM={int(vd)}"]
@@ -271,7 +282,8 @@ def load_host_module():
     return _HOST
 
 
-def build_all(head_dims=(16, 32, 48, 64, 128), latent_sizes=((64, 32), (512, 64)), capped_sizes=((64, 64), (32, 48))) -> None:
+def build_all(head_dims=(16, 32, 48, 64, 128), latent_sizes=((64, 32), (512, 64)), capped_sizes=((64, 64), (32, 48)),
+              ssd_sizes=((64, 32), (128, 64))) -> None:
     """Everything, for a build check."""
     host_module_path()
     for name in KERNEL_LIBS:
@@ -282,3 +294,5 @@ def build_all(head_dims=(16, 32, 48, 64, 128), latent_sizes=((64, 32), (512, 64)
         kernel_lib_path(latent_attention_lib_name(rank, rot))
     for kd, vd in capped_sizes:
         kernel_lib_path(capped_attention_lib_name(kd, vd))
+    for n, p in ssd_sizes:
+        kernel_lib_path(ssd_lib_name(n, p))

@@ -274,6 +274,29 @@ __device__ __forceinline__ float block_sum(float v, float* part) {
   return gb::warp_sum(t);
 }
 
+// out = tanh(alpha * x) * w + b per channel: a norm without statistics. grid (ceil(d / (4 * threads)), rows): a thread
+// takes four neighbouring channels of one row (VEC: rows start on 16 bytes and d is a multiple of four).
+template <typename OT, bool VEC>
+__global__ void __launch_bounds__(256)
+dynamic_tanh_kernel(const float* __restrict__ x, float alpha, const float* __restrict__ w, const float* __restrict__ b,
+                    OT* __restrict__ out, const int32_t* __restrict__ rows, int d) {
+  gb::pdl_launch_dependents();
+  gb::pdl_wait();
+  const size_t r = blockIdx.y;
+  const float* xr = x + (size_t)(rows ? rows[r] : r) * d;
+  OT* o = out + r * d;
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (c >= d) return;
+  if (VEC) {
+    const float4 v = *reinterpret_cast<const float4*>(xr + c);
+    const float4 ww = *reinterpret_cast<const float4*>(w + c), bb = *reinterpret_cast<const float4*>(b + c);
+    store4<OT>(o + c, fmaf(tanhf(alpha * v.x), ww.x, bb.x), fmaf(tanhf(alpha * v.y), ww.y, bb.y),
+               fmaf(tanhf(alpha * v.z), ww.z, bb.z), fmaf(tanhf(alpha * v.w), ww.w, bb.w));
+  } else {
+    for (int j = c; j < c + 4 && j < d; ++j) o[j] = gb::from_float<OT>(fmaf(tanhf(alpha * xr[j]), w[j], b[j]));
+  }
+}
+
 // out = (x - mean) / sqrt(var + eps) * w + b, var the mean of the squared deviations (taken in a
 // second pass over the row, not as mean(x^2) - mean^2). One block per row, 32-bit throughout.
 template <typename WT, typename OT>
@@ -552,6 +575,21 @@ GB_EXPORT int gb_layernorm(const float* x, const void* w, const void* b, int w_d
                                                  stream, dim3(1, 1, 1), x, (const WT*)w, (const WT*)b, eps, (OT*)out,
                                                  rows, d), "layernorm");
     });
+  });
+}
+
+// out[r] = tanh(alpha * x[row]) * w + b; rows (or null): which rows of x.
+GB_EXPORT int gb_dynamic_tanh(const float* x, float alpha, const float* w, const float* b, void* out, int out_dtype,
+                              const int32_t* rows, int n_rows, int d, cudaStream_t stream) {
+  if (n_rows <= 0 || d <= 0) return GB_OK;
+  if (n_rows > 65535) return gb::fail(GB_UNSUPPORTED, "dynamic_tanh: %d rows (at most 65535 a call)", n_rows);
+  const bool vec = d % 4 == 0 && (((uintptr_t)x | (uintptr_t)w | (uintptr_t)b | (uintptr_t)out) & 15) == 0;
+  const int quads = (d + 3) / 4, threads = quads >= 256 ? 256 : (quads + 31) / 32 * 32;
+  const dim3 grid((quads + threads - 1) / threads, n_rows);
+  return GB_DISPATCH_DTYPE(out_dtype, OT, [&]() -> int {
+    auto kernel = vec ? dynamic_tanh_kernel<OT, true> : dynamic_tanh_kernel<OT, false>;
+    return gb::check_pdl_launch(gb::launch_pdl(kernel, grid, dim3(threads), 0, stream, dim3(1, 1, 1), x, alpha, w, b, (OT*)out, rows, d),
+                                "dynamic_tanh");
   });
 }
 

@@ -113,7 +113,9 @@ struct EpilogueArgs {
 enum GateAct : int { GATE_SILU = 0, GATE_GELU_TANH = 1, GATE_CLAMPED_SWISH = 2,
                      // of one value, in the storing epilogue (EPI_STORE | EPI_GENERAL, bfloat16 out): relu(z)^2, tanh(z)
                      // xIELU: a z^2 + z / 2 for z > 0, b (exp(z) - 1 - z) + z / 2 for z <= 0, a = gate_limit, b = act_second
-                     STORE_RELU2 = 3, STORE_TANH = 4, STORE_XIELU = 5 };
+                     STORE_RELU2 = 3, STORE_TANH = 4, STORE_XIELU = 5,
+                     // the exact gelu, z (1 + erf(z / sqrt 2)) / 2
+                     STORE_GELU = 6 };
 
 // This CTA's slice of `bytes` at `base` into L2 (cta of ctas; 16-byte granules), by one thread.
 __device__ __forceinline__ void prefetch_slice_l2(const uint8_t* base, long long bytes, int cta, int ctas) {
@@ -239,6 +241,7 @@ __device__ __forceinline__ float store_act_fast(const EpilogueArgs& ra, float z)
     const float half = 0.5f * z;
     return z > 0.f ? fmaf(ra.gate_limit * z, z, half) : fmaf(ra.act_second, __expf(z) - 1.0f - z, half);
   }
+  if (ra.gate_act == STORE_GELU) return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
   return 1.0f - 2.0f * __frcp_rn(__expf(2.0f * z) + 1.0f);
 }
 
@@ -1628,7 +1631,7 @@ GB_EXPORT int gb_gemm_tc_supported(const void* x, const void* w, int Mx, int Nw,
 // 2: w holds gate and up rows packed in groups of 64 ([128 * ceil(Nw / 64), K], see the head of this
 // file); out[Mx,Nw] (bf16) = act(x gate^T, x up^T), act by gate_act: silu(g) u unless told otherwise.
 // alpha: the accumulating epilogue adds alpha * product. gate_act, gate_limit: the gated epilogue's
-// activation (GateAct), or with epi 0 and a bfloat16 output STORE_RELU2 / STORE_TANH / STORE_XIELU: out =
+// activation (GateAct), or with epi 0 and a bfloat16 output STORE_RELU2 / STORE_TANH / STORE_XIELU / STORE_GELU: out =
 // act(x w^T); act_second: the second number of an activation that has two (STORE_XIELU).
 GB_EXPORT int gb_gemm_tc(const void* x, const void* w, void* out, int Mx, int Nw, int K, int out_dtype, int epi,
                          const GbNormFold* norm, float alpha, int gate_act, float gate_limit, float act_second,
@@ -1643,7 +1646,7 @@ GB_EXPORT int gb_gemm_tc(const void* x, const void* w, void* out, int Mx, int Nw
   EpilogueArgs ra{};
   fold_norm(ra, norm);
   take_next_stream(ra);
-  if (gate_act < GATE_SILU || gate_act > STORE_XIELU) return gb::fail(GB_BAD_ARGUMENT, "gemm_tc: activation %d", gate_act);
+  if (gate_act < GATE_SILU || gate_act > STORE_GELU) return gb::fail(GB_BAD_ARGUMENT, "gemm_tc: activation %d", gate_act);
   if (gate_act >= STORE_RELU2 && ((epi & 7) != EPI_STORE || out_dtype != GB_BF16))
     return gb::fail(GB_BAD_ARGUMENT, "gemm_tc: an activation of one value goes with the storing epilogue and a bfloat16 output");
   if (gate_act < STORE_RELU2 && (epi & 7) != EPI_SWIGLU) gate_act = GATE_SILU;       // means nothing to the other epilogues
@@ -1707,7 +1710,10 @@ GB_EXPORT int gb_gemm_tc_grouped(const void* x, const void* w, void* out, int Mx
   if (epi != EPI_STORE && epi != EPI_SWIGLU) return gb::fail(GB_UNSUPPORTED, "gemm_tc_grouped: epilogue %d", epi);
   if (epi == EPI_SWIGLU && out_dtype != GB_BF16)
     return gb::fail(GB_BAD_ARGUMENT, "gemm_tc_grouped: the gated epilogue writes bfloat16");
-  if (gate_act < GATE_SILU || gate_act > GATE_CLAMPED_SWISH) return gb::fail(GB_BAD_ARGUMENT, "gemm_tc_grouped: gate activation %d", gate_act);
+  if (gate_act < GATE_SILU || gate_act > STORE_GELU || gate_act == STORE_XIELU)
+    return gb::fail(GB_BAD_ARGUMENT, "gemm_tc_grouped: activation %d", gate_act);
+  if (gate_act >= STORE_RELU2 && (epi != EPI_STORE || out_dtype != GB_BF16))
+    return gb::fail(GB_BAD_ARGUMENT, "gemm_tc_grouped: an activation of one value goes with the storing epilogue and a bfloat16 output");
   const int weight_rows = epi == EPI_SWIGLU ? 128 * ((Nw + 63) / 64) : Nw;
   if ((long long)groups * weight_rows > 0x7fffffffLL) return gb::fail(GB_UNSUPPORTED, "gemm_tc_grouped: too many weight rows");
   EpilogueArgs ra{};
@@ -1726,6 +1732,8 @@ GB_EXPORT int gb_gemm_tc_grouped(const void* x, const void* w, void* out, int Mx
       return launch_persistent<BN_, EPI_SWIGLU | EPI_GENERAL, __nv_bfloat16>(mm, mn, (__nv_bfloat16*)out, Nw, Mx, weight_rows, Nw, K, stream, ra); \
     if (epi == EPI_SWIGLU)                                                                                            \
       return launch_persistent<BN_, EPI_SWIGLU, __nv_bfloat16>(mm, mn, (__nv_bfloat16*)out, Nw, Mx, weight_rows, Nw, K, stream, ra); \
+    if (gate_act >= STORE_RELU2)                                                                                      \
+      return launch_persistent<BN_, EPI_STORE | EPI_GENERAL, __nv_bfloat16>(mm, mn, (__nv_bfloat16*)out, Nw, Mx, weight_rows, Nw, K, stream, ra); \
     if (out_dtype == GB_F32)                                                                                          \
       return launch_persistent<BN_, EPI_STORE, float>(mm, mn, (float*)out, Nw, Mx, weight_rows, Nw, K, stream, ra);   \
     return launch_persistent<BN_, EPI_STORE, __nv_bfloat16>(mm, mn, (__nv_bfloat16*)out, Nw, Mx, weight_rows, Nw, K, stream, ra); \

@@ -91,6 +91,39 @@ __device__ __forceinline__ float gate_act(int kind, float limit, float g, float 
   return (g / (1.0f + expf(-g))) * u;
 }
 
+// an activation of one value, for experts without a gate
+__device__ __forceinline__ float plain_act(int kind, float z) {
+  switch (kind) {
+    case 0: return 1.0f / (1.0f + expf(-z));
+    case 1: return z / (1.0f + expf(-z));
+    case 2: return fmaxf(z, 0.f) * fmaxf(z, 0.f);
+    case 3: return tanhf(z);
+    default: return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
+  }
+}
+
+// grid (T, top). act[(t * top + j)][f] = act(up_e[f] . h_t), e = ids[t][j], the expert's weights [F, K]; a warp
+// per feature, lanes over k. in_scale as below.
+template <typename HT, typename WT, typename OT>
+__global__ void __launch_bounds__(128)
+moe_up_kernel(const HT* __restrict__ h, const WT* __restrict__ w, const int32_t* __restrict__ ids, OT* __restrict__ act,
+              int top, int F, int K, int kind, const float* __restrict__ in_scale) {
+  extern __shared__ float h_s[];
+  const int t = blockIdx.x, j = blockIdx.y;
+  for (int k = threadIdx.x; k < K; k += blockDim.x) h_s[k] = gb::to_float<HT>(h[(size_t)t * K + k]);
+  __syncthreads();
+  const float s_in = in_scale ? in_scale[(size_t)t * top + j] : 1.0f;
+  const WT* we = w + (size_t)ids[(size_t)t * top + j] * F * K;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int f = warp; f < F; f += 4) {
+    const WT* ur = we + (size_t)f * K;
+    float u = 0.f;
+    for (int k = lane; k < K; k += 32) u = fmaf(h_s[k], gb::to_float<WT>(ur[k]), u);
+    u = gb::warp_sum(u) * s_in;
+    if (lane == 0) act[((size_t)t * top + j) * F + f] = gb::from_float<OT>(plain_act(kind, u));
+  }
+}
+
 // grid (T, top). act[(t * top + j)][f] = act(gate_e[f] . h_t, up_e[f] . h_t), e = ids[t][j]; the
 // expert's weights are [2F, K]: F gate rows, then F up rows. A warp per feature, lanes over k.
 // in_scale [T, top] (or null): the pair's factor on the expert's input, expert(s h): both products
@@ -180,6 +213,23 @@ GB_EXPORT int gb_moe_gate_up(const void* h, int h_dtype, const void* w, int w_dt
         moe_gate_up_kernel<HT, WT, OT><<<dim3(T, top), 128, (size_t)K * sizeof(float), stream>>>(
             (const HT*)h, (const WT*)w, ids, (OT*)act, top, F, K, kind, limit, in_scale);
         return gb::check_launch("moe_gate_up");
+      });
+    });
+  });
+}
+
+// kind: 0 sigmoid, 1 silu, 2 relu^2, 3 tanh, 4 exact gelu.
+GB_EXPORT int gb_moe_up(const void* h, int h_dtype, const void* w, int w_dtype, const int32_t* ids, void* act, int act_dtype,
+                        int T, int top, int F, int K, int kind, const float* in_scale, cudaStream_t stream) {
+  if (T <= 0) return GB_OK;
+  if (kind < 0 || kind > 4) return gb::fail(GB_BAD_ARGUMENT, "moe_up: activation %d", kind);
+  if ((size_t)K * sizeof(float) > 48 * 1024) return gb::fail(GB_UNSUPPORTED, "moe_up: width %d", K);
+  return GB_DISPATCH_DTYPE(h_dtype, HT, [&]() -> int {
+    return GB_DISPATCH_DTYPE(w_dtype, WT, [&]() -> int {
+      return GB_DISPATCH_DTYPE(act_dtype, OT, [&]() -> int {
+        moe_up_kernel<HT, WT, OT><<<dim3(T, top), 128, (size_t)K * sizeof(float), stream>>>(
+            (const HT*)h, (const WT*)w, ids, (OT*)act, top, F, K, kind, in_scale);
+        return gb::check_launch("moe_up");
       });
     });
   });

@@ -77,16 +77,30 @@ __device__ __forceinline__ float gate_act(int kind, float limit, float g, float 
   return (g / (1.0f + expf(-g))) * u;
 }
 
+// an activation of one value, for experts without a gate (ACT_UP below)
+__device__ __forceinline__ float plain_act(int kind, float z) {
+  switch (kind) {
+    case 0: return 1.0f / (1.0f + expf(-z));
+    case 1: return z / (1.0f + expf(-z));
+    case 2: return fmaxf(z, 0.f) * fmaxf(z, 0.f);
+    case 3: return tanhf(z);
+    default: return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
+  }
+}
+
+// What a grouped product does with its sums: store them, act(gate, up) of two products, act(up) of one.
+enum GroupedMode : int { PLAIN = 0, GATED_UP = 1, ACT_UP = 2 };
+
 // out[row0 + r][n] = sum_k A_e[r][k] * W_e[n][k] for the tile's rows r and columns n0 .. n0 + 63.
 // A_e's row r is a[e * a_group + (gather ? gather[row0 + r] / gather_div : row0 + r) * lda ..];
-// out's row is out[e * out_group + (row0 + r) * ldo ..]. GATED: W_e has N gate rows followed by N up
+// out's row is out[e * out_group + (row0 + r) * ldo ..]. GATED_UP: W_e has N gate rows followed by N up
 // rows (or the packed layout, see `packed`), and out (bfloat16) is act(gate, up). With a tile list (tile_expert ...) the CTA reads its
 // group and rows from it; without, blockIdx.z is the group and every group has `rows_all` rows.
 // The CTA is WM x WN warps, a warp's tile (MI * 16) x (NP * 16): 128 x 64 for groups of many rows,
-// 16 x 64 for a few rows per group, where a taller tile would be padding. GATED with in_scale: the
+// 16 x 64 for a few rows per group, where a taller tile would be padding. With in_scale (GATED_UP, ACT_UP): the
 // products of row r are multiplied by in_scale[gather[row0 + r]] before the activation (a factor on
 // the expert's input, in which both products are linear).
-template <int WM, int WN, int MI, int NP, bool GATED, typename OT>
+template <int WM, int WN, int MI, int NP, int MODE, typename OT>
 __global__ void __launch_bounds__(WM * WN * 32)
 grouped_gemm_kernel(const __nv_bfloat16* __restrict__ a, int lda, long long a_group, const int32_t* __restrict__ gather,
                     int gather_div, const __nv_bfloat16* __restrict__ w, long long w_group, OT* __restrict__ out, int ldo,
@@ -94,6 +108,7 @@ grouped_gemm_kernel(const __nv_bfloat16* __restrict__ a, int lda, long long a_gr
                     const int32_t* __restrict__ tile_row0, const int32_t* __restrict__ tile_rows,
                     const int32_t* __restrict__ num_tiles, int rows_all, int kind, float limit, int packed,
                     const float* __restrict__ in_scale) {
+  constexpr bool GATED = MODE == GATED_UP, SCALED = MODE != PLAIN;
   constexpr int TM = WM * MI * 16, TN = WN * NP * 16, THREADS = WM * WN * 32;
   constexpr int BROWS = GATED ? 2 * TN : TN;
   constexpr int CH = GK / 8;                       // 16-byte chunks of a tile's row
@@ -101,7 +116,7 @@ grouped_gemm_kernel(const __nv_bfloat16* __restrict__ a, int lda, long long a_gr
   auto a_tile = [&](int stage) { return tiles + (size_t)stage * (TM + BROWS) * GPITCH; };
   auto b_tile = [&](int stage) { return tiles + ((size_t)stage * (TM + BROWS) + TM) * GPITCH; };
   __shared__ int32_t src_row[TM];
-  __shared__ float row_scale[GATED ? TM : 1];
+  __shared__ float row_scale[SCALED ? TM : 1];
   int e, row0, rows;
   if (tile_expert != nullptr) {
     const int tile = blockIdx.y;
@@ -115,7 +130,7 @@ grouped_gemm_kernel(const __nv_bfloat16* __restrict__ a, int lda, long long a_gr
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   for (int r = tid; r < TM; r += THREADS)
     src_row[r] = r < rows ? (gather ? gather[row0 + r] / gather_div : row0 + r) : -1;
-  if (GATED)
+  if (SCALED)
     for (int r = tid; r < TM; r += THREADS)
       row_scale[r] = (in_scale != nullptr && gather != nullptr && r < rows) ? in_scale[gather[row0 + r]] : 1.0f;
   __syncthreads();
@@ -206,6 +221,7 @@ grouped_gemm_kernel(const __nv_bfloat16* __restrict__ a, int lda, long long a_gr
         if (r >= rows || n >= N) continue;
         float v = acc[mi][nt][x];
         if (GATED) v = gate_act(kind, limit, v * row_scale[GATED ? r : 0], acc_u[GATED ? mi : 0][nt][x] * row_scale[GATED ? r : 0]);
+        if (MODE == ACT_UP) v = plain_act(kind, v * row_scale[SCALED ? r : 0]);
         oe[(size_t)(row0 + r) * ldo + n] = gb::from_float<OT>(v);
       }
 }
@@ -226,12 +242,12 @@ moe_combine_kernel(const float* __restrict__ y, const int32_t* __restrict__ pair
 }
 
 
-template <int WM, int WN, int MI, int NP, bool GATED, typename OT, typename... Args>
+template <int WM, int WN, int MI, int NP, int MODE, typename OT, typename... Args>
 int launch_grouped(dim3 grid, cudaStream_t stream, const char* what, Args... args) {
   constexpr int TM = WM * MI * 16, TN = WN * NP * 16;
-  constexpr size_t smem = (size_t)STAGES * (TM + (GATED ? 2 * TN : TN)) * GPITCH;
+  constexpr size_t smem = (size_t)STAGES * (TM + (MODE == GATED_UP ? 2 * TN : TN)) * GPITCH;
   static gb::OncePerDevice attribute;
-  auto kernel = grouped_gemm_kernel<WM, WN, MI, NP, GATED, OT>;
+  auto kernel = grouped_gemm_kernel<WM, WN, MI, NP, MODE, OT>;
   if (smem > 48 * 1024 && attribute.needed()) {
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return gb::fail(GB_CUDA_ERROR, "%s: %s", what, cudaGetErrorString(e));
@@ -249,16 +265,19 @@ GB_EXPORT long long gb_moe_grouped_index_words(long long R, int E) {
   return 2 * R + 3 * tiles + 4;
 }
 
-// h [T, K], w_gate_up [E, 2F, K] (packed: [E, 128 * ceil(F / 64), K], gate and up rows in groups of 64),
+// h [T, K], w_gate_up by layout: 0 [E, 2F, K] (gate rows, then up rows), 1 [E, 128 * ceil(F / 64), K] (gate and up
+// rows in groups of 64), 2 [E, F, K] (experts without a gate: act(up h), kind as for gb_moe_up),
 // w_down [E, N, F] bfloat16; ids [T, top], weights [T, top]; x [T, N] 32-bit.
 // index: gb_moe_grouped_index_words int32; act: [T * top, F] bfloat16; y: [T * top, N] 32-bit.
 GB_EXPORT int gb_moe_grouped(const void* h, const void* w_gate_up, const void* w_down, const int32_t* ids,
                              const float* weights, float* x, int T, int top, int E, int F, int K, int N, int kind,
-                             float limit, float alpha, int packed, int scale_input, int32_t* index, void* act, float* y,
+                             float limit, float alpha, int layout, int scale_input, int32_t* index, void* act, float* y,
                              cudaStream_t stream) {
   if (T <= 0) return GB_OK;
   if (K % 8 || F % 8) return gb::fail(GB_UNSUPPORTED, "moe_grouped: widths %d and %d must be multiples of 8", K, F);
   if (E < 1 || (size_t)E * 2 * sizeof(int32_t) > 40 * 1024) return gb::fail(GB_UNSUPPORTED, "moe_grouped: %d experts", E);
+  if (layout < 0 || layout > 2) return gb::fail(GB_BAD_ARGUMENT, "moe_grouped: layout %d", layout);
+  const int packed = layout == 1;
   const long long R = (long long)T * top;
   const bool tall = R >= 48LL * E;             // on average 48 rows an expert or more
   const int gm = tall ? TALL : SHORT;
@@ -284,20 +303,26 @@ GB_EXPORT int gb_moe_grouped(const void* h, const void* w_gate_up, const void* w
   const float* in_scale = scale_input ? weights : nullptr;       // the weights scale what goes into an expert ...
   const float* out_weights = scale_input ? nullptr : weights;    // ... or what comes out of it
   const float* no_scale = nullptr;
-  const long long zero = 0, gu_group = (long long)(packed ? 128 * ((F + 63) / 64) : 2 * F) * K, d_group = (long long)N * F;
-  if (tall)
-    rc = launch_grouped<4, 2, 2, 2, true, __nv_bfloat16>(grid_f, stream, "moe_gate_up_grouped", hh, K, zero, rp, top, wgu,
+  const long long zero = 0, gu_group = (long long)(layout == 1 ? 128 * ((F + 63) / 64) : layout == 0 ? 2 * F : F) * K, d_group = (long long)N * F;
+  if (layout == 2 && tall)
+    rc = launch_grouped<4, 2, 2, 2, ACT_UP, __nv_bfloat16>(grid_f, stream, "moe_up_grouped", hh, K, zero, rp, top, wgu, gu_group,
+                                                          a, F, zero, F, K, te, t0, tr, nt, 0, kind, limit, 0, in_scale);
+  else if (layout == 2)
+    rc = launch_grouped<1, 4, 1, 1, ACT_UP, __nv_bfloat16>(grid_f, stream, "moe_up_grouped", hh, K, zero, rp, top, wgu, gu_group,
+                                                          a, F, zero, F, K, te, t0, tr, nt, 0, kind, limit, 0, in_scale);
+  else if (tall)
+    rc = launch_grouped<4, 2, 2, 2, GATED_UP, __nv_bfloat16>(grid_f, stream, "moe_gate_up_grouped", hh, K, zero, rp, top, wgu,
                                                         gu_group, a, F, zero, F, K, te, t0, tr, nt, 0, kind, limit, packed, in_scale);
   else
-    rc = launch_grouped<1, 4, 1, 1, true, __nv_bfloat16>(grid_f, stream, "moe_gate_up_grouped", hh, K, zero, rp, top, wgu,
+    rc = launch_grouped<1, 4, 1, 1, GATED_UP, __nv_bfloat16>(grid_f, stream, "moe_gate_up_grouped", hh, K, zero, rp, top, wgu,
                                                         gu_group, a, F, zero, F, K, te, t0, tr, nt, 0, kind, limit, packed, in_scale);
   if (rc != GB_OK) return rc;
   const __nv_bfloat16* ac = a;
   if (tall)
-    rc = launch_grouped<4, 2, 2, 2, false, float>(grid_n, stream, "moe_down_grouped", ac, F, zero, none, 1, wd, d_group, y, N,
+    rc = launch_grouped<4, 2, 2, 2, PLAIN, float>(grid_n, stream, "moe_down_grouped", ac, F, zero, none, 1, wd, d_group, y, N,
                                                  zero, N, F, te, t0, tr, nt, 0, 0, 0.f, 0, no_scale);
   else
-    rc = launch_grouped<1, 4, 1, 1, false, float>(grid_n, stream, "moe_down_grouped", ac, F, zero, none, 1, wd, d_group, y, N,
+    rc = launch_grouped<1, 4, 1, 1, PLAIN, float>(grid_n, stream, "moe_down_grouped", ac, F, zero, none, 1, wd, d_group, y, N,
                                                  zero, N, F, te, t0, tr, nt, 0, 0, 0.f, 0, no_scale);
   if (rc != GB_OK) return rc;
   moe_combine_kernel<<<T, 256, 0, stream>>>(y, pair_row, out_weights, x, top, N, alpha);
@@ -417,10 +442,10 @@ GB_EXPORT int gb_grouped_gemm(const void* a, int lda, long long a_group, const v
   __nv_bfloat16* oo = (__nv_bfloat16*)out;
   const int32_t* none = nullptr;
   if (M >= 48)
-    return launch_grouped<4, 2, 2, 2, false, __nv_bfloat16>(dim3((N + GN - 1) / GN, (M + TALL - 1) / TALL, groups), stream,
+    return launch_grouped<4, 2, 2, 2, PLAIN, __nv_bfloat16>(dim3((N + GN - 1) / GN, (M + TALL - 1) / TALL, groups), stream,
                                                            "grouped_gemm", aa, lda, a_group, none, 1, ww, w_group, oo, ldo,
                                                            out_group, N, K, none, none, none, none, M, 0, 0.f, 0, (const float*)nullptr);
-  return launch_grouped<1, 4, 1, 1, false, __nv_bfloat16>(dim3((N + GN - 1) / GN, (M + SHORT - 1) / SHORT, groups), stream,
+  return launch_grouped<1, 4, 1, 1, PLAIN, __nv_bfloat16>(dim3((N + GN - 1) / GN, (M + SHORT - 1) / SHORT, groups), stream,
                                                          "grouped_gemm", aa, lda, a_group, none, 1, ww, w_group, oo, ldo,
                                                          out_group, N, K, none, none, none, none, M, 0, 0.f, 0, (const float*)nullptr);
 }

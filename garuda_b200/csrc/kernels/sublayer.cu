@@ -4,9 +4,10 @@
 //   qk_norm_rope_append  a projected row -> queries (RMS norm per head with a weight per head and
 //                        channel, rotation of the first channels) to q_out; keys (the same, one
 //                        weight for all heads) and values into their pages; the values may be the
-//                        keys' own columns as projected (before norm and rotation)
+//                        keys' own columns as projected (before norm and rotation); queries may also be
+//                        multiplied by a number that grows with their position
 //   gate_mul             x <- x * act(gate), act = sigmoid | silu, the gate's logits 32-bit
-//   unary_act            out = act(z), act = relu^2 | tanh
+//   unary_act            out = act(z), act = sigmoid | silu | relu^2 | tanh | exact gelu
 //   sublayer_merge       y = alpha * sum_b rms(y_b) * w_b   (or y = y_0)
 //                        y <- y * sigmoid(gate + bias)      (optional)
 //                        x <- x + rms(y) * w                (or out = y)
@@ -27,7 +28,7 @@ qk_norm_rope_append_kernel(const float* __restrict__ src, int row_stride, int q_
                            const int32_t* __restrict__ positions, const int32_t* __restrict__ token_req,
                            const int32_t* __restrict__ block_table, int table_width, int Hq, int Hkv, int dim, int vdim,
                            const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
-                           const float* __restrict__ inv_freq, int interleaved, int page_size) {
+                           const float* __restrict__ inv_freq, int interleaved, int page_size, float q_coef, int q_every) {
   __shared__ float sin_s[QK_MAX_DIM / 2], cos_s[QK_MAX_DIM / 2];
   gb::pdl_launch_dependents();
   gb::pdl_wait();
@@ -45,8 +46,10 @@ qk_norm_rope_append_kernel(const float* __restrict__ src, int row_stride, int q_
   __syncthreads();
   const float* row = src + (size_t)t * row_stride;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  // what the token's queries are multiplied by (q_every 0: nothing)
+  const float growth = q_every > 0 ? fmaf(q_coef, logf((float)((pos + 1) / q_every + 1)), 1.0f) : 1.0f;
   // every head of the row starts on 8 bytes (the head width is even)
-  const bool paired = interleaved && ((row_stride | q_col | k_col) & 1) == 0 && (reinterpret_cast<uintptr_t>(src) & 7) == 0 &&
+  const bool paired = (interleaved || !rotate) && ((row_stride | dim | q_col | k_col) & 1) == 0 && (reinterpret_cast<uintptr_t>(src) & 7) == 0 &&
                       ((reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(k_pool)) & (2 * sizeof(OT) - 1)) == 0;
   for (int head = warp; head < Hq + Hkv; head += warps) {
     const bool is_q = head < Hq;
@@ -60,6 +63,7 @@ qk_norm_rope_append_kernel(const float* __restrict__ src, int row_stride, int q_
       for (int c = lane; c < dim; c += 32) ss = fmaf(s[c], s[c], ss);
       inv = 1.0f / sqrtf(gb::warp_sum(ss) / (float)dim + eps);
     }
+    const float times = is_q ? growth : 1.0f;
     OT* dst = is_q ? q_out + ((size_t)t * Hq + head) * dim
                    : k_pool + ((cache_row + (head - Hq)) * page_size + (pos % page_size)) * dim;
     if (paired) {        // neighbours rotate together: one 8-byte load and one store for the two
@@ -71,7 +75,7 @@ qk_norm_rope_append_kernel(const float* __restrict__ src, int row_stride, int q_
           const float ra = a * cos_s[i] - b * sin_s[i], rb = b * cos_s[i] + a * sin_s[i];
           a = ra, b = rb;
         }
-        gb::store_pair(dst + 2 * i, a, b);
+        gb::store_pair(dst + 2 * i, a * times, b * times);
       }
       continue;
     }
@@ -84,8 +88,13 @@ qk_norm_rope_append_kernel(const float* __restrict__ src, int row_stride, int q_
         const float ra = a * cos_s[i] - b * sin_s[i], rb = b * cos_s[i] + a * sin_s[i];
         a = ra, b = rb;
       }
-      dst[ia] = gb::from_float<OT>(a);
-      dst[ib] = gb::from_float<OT>(b);
+      dst[ia] = gb::from_float<OT>(a * times);
+      dst[ib] = gb::from_float<OT>(b * times);
+    }
+    if ((dim & 1) && lane == 0) {          // the last channel of an odd head has no partner (and no rotation)
+      float a = s[dim - 1];
+      if (normed) a = (a * inv) * w[dim - 1];
+      dst[dim - 1] = gb::from_float<OT>(a * times);
     }
   }
   if (cache_row >= 0) {
@@ -97,13 +106,14 @@ qk_norm_rope_append_kernel(const float* __restrict__ src, int row_stride, int q_
   }
 }
 
-enum { ACT_SIGMOID = 0, ACT_SILU = 1, ACT_RELU2 = 2, ACT_TANH = 3 };
+enum { ACT_SIGMOID = 0, ACT_SILU = 1, ACT_RELU2 = 2, ACT_TANH = 3, ACT_GELU = 4 };
 
 __device__ __forceinline__ float act(float z, int kind) {
   switch (kind) {
     case ACT_SIGMOID: return sigmoidf_(z);
     case ACT_SILU: return z * sigmoidf_(z);
     case ACT_RELU2: { const float r = fmaxf(z, 0.f); return r * r; }
+    case ACT_GELU: return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
     default: return tanhf(z);
   }
 }
@@ -290,9 +300,10 @@ GB_EXPORT int gb_qk_norm_rope_append(const float* src, int row_stride, int q_col
                                      void* k_pool, void* v_pool, int out_dtype, const int32_t* positions,
                                      const int32_t* token_req, const int32_t* block_table, int table_width, int T, int Hq,
                                      int Hkv, int dim, int vdim, const float* q_w, const float* k_w, float eps,
-                                     const float* inv_freq, int interleaved, int page_size, cudaStream_t stream) {
+                                     const float* inv_freq, int interleaved, int page_size, float q_coef, int q_every,
+                                     cudaStream_t stream) {
   if (T <= 0) return GB_OK;
-  if (dim % 2 || dim > QK_MAX_DIM) return gb::fail(GB_UNSUPPORTED, "qk_norm_rope_append: head width %d (even, at most %d)", dim, QK_MAX_DIM);
+  if (inv_freq != nullptr && (dim % 2 || dim > QK_MAX_DIM)) return gb::fail(GB_UNSUPPORTED, "qk_norm_rope_append: a rotated head of %d channels (even, at most %d)", dim, QK_MAX_DIM);
   if (Hkv > 0 && (!k_pool || !v_pool || !block_table || page_size < 1))
     return gb::fail(GB_BAD_ARGUMENT, "qk_norm_rope_append: kv heads given without a cache to store them in");
   const int heads = Hq + Hkv;
@@ -301,7 +312,7 @@ GB_EXPORT int gb_qk_norm_rope_append(const float* src, int row_stride, int q_col
     return gb::check_pdl_launch(
         gb::launch_pdl(qk_norm_rope_append_kernel<OT>, dim3(T), dim3(block), 0, stream, dim3(1, 1, 1), src, row_stride, q_col,
                        k_col, v_col, (OT*)q_out, (OT*)k_pool, (OT*)v_pool, positions, token_req, block_table, table_width, Hq,
-                       Hkv, dim, vdim, q_w, k_w, eps, inv_freq, interleaved, page_size),
+                       Hkv, dim, vdim, q_w, k_w, eps, inv_freq, interleaved, page_size, q_coef, q_every),
         "qk_norm_rope_append");
   });
 }
@@ -323,7 +334,7 @@ GB_EXPORT int gb_gate_mul(void* x, int x_dtype, const float* gate, int gate_stri
 GB_EXPORT int gb_unary_act(const void* z, int z_dtype, int z_stride, void* out, int out_dtype, int out_stride, int T, int n,
                            int kind, cudaStream_t stream) {
   if (T <= 0 || n <= 0) return GB_OK;
-  if (kind < ACT_SIGMOID || kind > ACT_TANH) return gb::fail(GB_BAD_ARGUMENT, "unary_act: kind %d", kind);
+  if (kind < ACT_SIGMOID || kind > ACT_GELU) return gb::fail(GB_BAD_ARGUMENT, "unary_act: kind %d", kind);
   if (T > 65535) return gb::fail(GB_UNSUPPORTED, "unary_act: %d rows (at most 65535 a call)", T);
   const dim3 grid((n + 1023) / 1024, T);
   return GB_DISPATCH_DTYPE(z_dtype, IT, [&]() -> int {

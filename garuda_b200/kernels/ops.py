@@ -89,6 +89,7 @@ class CudaOps:
         self._mixers = None
         self._state = None
         self._seq = None
+        self._ssd = None
         self._declare_core()
         # A word of pinned host memory that a kernel whose bounded wait ran out writes its code to (the
         # device reaches pinned host memory directly); ``failed_wait`` reads it without a copy.
@@ -122,6 +123,7 @@ class CudaOps:
             "gb_embedding_copies": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
             "gb_scale_softcap": [c_void_p, c_longlong, c_float, c_float, c_void_p],
             "gb_layernorm": [c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
+            "gb_dynamic_tanh": [c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p],
             "gb_residual_axpy": [c_void_p, c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_int, c_void_p],
             "gb_rms_add": [c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_int, c_int, c_void_p],
             "gb_gelu_gather_mul": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
@@ -199,6 +201,30 @@ class CudaOps:
             self._seq = L
         return self._seq
 
+    @property
+    def ssd_lib(self):
+        """The library of the state-space kernels, compiled and loaded when a model first needs it."""
+        if self._ssd is None:
+            L = load_kernel_lib("garuda_ssd")
+            L.gb_last_error.restype = ctypes.c_char_p
+            for name, argtypes in self._SSD_SIGNATURES.items():
+                fn = getattr(L, name)
+                fn.argtypes = argtypes
+                fn.restype = c_int
+            self._ssd = L
+        return self._ssd
+
+    _SSD_SIGNATURES = {
+        "gb_ssd_prepare": [c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p,
+                           c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "gb_ssd_recurrence": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int,
+                              c_int, c_int, c_void_p, c_void_p],
+        "gb_ssd_decode": [c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p,
+                          c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+        "gb_ssd_finish": [c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int,
+                          c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+    }
+
     _SEQ_SIGNATURES = {
         "gb_post_norm": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_void_p],
         "gb_group_gate_mul": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
@@ -239,7 +265,7 @@ class CudaOps:
                              c_void_p],
         "gb_qk_norm_rope_append": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                    c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
-                                   c_void_p, c_int, c_int, c_void_p],
+                                   c_void_p, c_int, c_int, c_float, c_int, c_void_p],
         "gb_gate_mul": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
         "gb_unary_act": [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "gb_sublayer_merge": [c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_int, c_void_p, c_void_p, c_float,
@@ -255,6 +281,8 @@ class CudaOps:
                               c_void_p, c_void_p],
             "gb_moe_gate_up": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                c_int, c_float, c_void_p, c_void_p],
+            "gb_moe_up": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                          c_void_p],
             "gb_moe_down": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                             c_float, c_void_p],
             "gb_moe_grouped": [c_void_p] * 6 + [c_int] * 7 + [c_float, c_float, c_int, c_int] + [c_void_p] * 4,
@@ -603,6 +631,20 @@ class CudaOps:
             x.data_ptr(), weight.data_ptr(), _ptr(bias), _tag(weight, "norm weight"), float(eps), out.data_ptr(),
             _tag(out, "layernorm out"), _ptr(rows), n, d, self._stream()), "layernorm")
 
+    def dynamic_tanh(self, x, alpha, weight, bias, out, rows=None):
+        """``out = tanh(alpha * x) * weight + bias`` per channel (x, weight, bias 32-bit), ``out`` in its
+        own dtype; ``rows``: only these rows of ``x``."""
+        self._on_device(x, weight, bias, out, rows)
+        _need(x.dtype == torch.float32 and x.is_contiguous() and x.dim() == 2, "dynamic_tanh: x must be float32 [T, d]")
+        d = x.shape[1]
+        _need(all(v.dtype == torch.float32 and v.is_contiguous() and v.numel() == d for v in (weight, bias)),
+              "dynamic_tanh: weight and bias float32 [d]")
+        n = x.shape[0] if rows is None else rows.shape[0]
+        _need(tuple(out.shape) == (n, d) and out.is_contiguous() and (rows is None or rows.dtype == torch.int32), "dynamic_tanh: out, rows")
+        self._check(self.core, self.core.gb_dynamic_tanh(
+            x.data_ptr(), float(alpha), weight.data_ptr(), bias.data_ptr(), out.data_ptr(), _tag(out, "dynamic_tanh out"), _ptr(rows), n,
+            d, self._stream()), "dynamic_tanh")
+
     def residual_axpy(self, x, y=None, alpha: float = 1.0, row=None):
         """``x[t] += alpha * y[t] + row`` on the 32-bit residual; ``y`` or ``row`` may be None."""
         self._on_device(x, y, row)
@@ -719,6 +761,19 @@ class CudaOps:
             act.data_ptr(), _tag(act, "act"), w_down.data_ptr(), _tag(w_down, "w"), ids.data_ptr(),
             _ptr(weights), x.data_ptr(), T, top, F, N, float(alpha), self._stream()), "moe_down")
 
+    def moe_up(self, h, w_up, ids, act, kind: str, in_scale=None):
+        """``act[T, top, F]``: as ``moe_gate_up`` for experts without a gate, ``w_up [E, F, K]``, an activation
+        of one value (``UNARY_ACTS``)."""
+        self._on_device(h, w_up, ids, act)
+        T, K = h.shape
+        top = ids.shape[1]
+        E, F, _ = w_up.shape
+        _need(h.is_contiguous() and w_up.is_contiguous() and act.is_contiguous() and h.dtype == w_up.dtype
+              and w_up.shape[2] == K and act.shape == (T, top, F), "moe_up: shapes")
+        self._check(self.mixers, self.mixers.gb_moe_up(
+            h.data_ptr(), _tag(h, "h"), w_up.data_ptr(), _tag(w_up, "w"), ids.data_ptr(), act.data_ptr(), _tag(act, "act"), T, top,
+            F, K, self.UNARY_ACTS[kind], _ptr(in_scale), self._stream()), "moe_up")
+
     def pack_expert_gate_up(self, gates, ups):
         """The experts' gate and up matrices stacked, in the layout ``routed_feed_forward`` wants:
         ``[E, 2F, K]`` (an expert's gate rows, then its up rows), or, where the tensor-core products
@@ -734,24 +789,26 @@ class CudaOps:
     GROUPED_TC_PAIRS = 1024
 
     def routed_feed_forward(self, ctx, h, w_gate_up, w_down, ids, weights, x, kind: str, limit: float,
-                            alpha: float = 1.0, scale_input: bool = False):
+                            alpha: float = 1.0, scale_input: bool = False, gated: bool = True):
         """``x[t] += alpha * sum_j weights[t, j] * expert_{ids[t, j]}(h[t])`` with the experts'
-        weights stacked: ``w_gate_up`` from ``pack_expert_gate_up``, ``w_down [E, N, F]``.
+        weights stacked: ``w_gate_up`` from ``pack_expert_gate_up``, ``w_down [E, N, F]``. Without ``gated``:
+        ``w_gate_up`` is ``[E, F, K]``, the up rows alone, and ``kind`` an activation of one value.
         ``scale_input``: the weight multiplies what goes into the expert instead,
         ``sum_j expert(weights[t, j] * h[t])``."""
         T, top = ids.shape
         E, N, F = w_down.shape
         K = h.shape[1]
         packed = getattr(w_gate_up, "gb_group", 0) == 64
-        if packed and T * top >= self.GROUPED_TC_PAIRS and self._routed_tcgen05(ctx, h, w_gate_up, w_down, ids, weights,
-                                                                               x, kind, limit, alpha, scale_input):
+        grouped = packed if gated else (self.tc is not None and h.dtype == torch.bfloat16 and K % 8 == 0 and F % 8 == 0 and E <= 4096)
+        if grouped and T * top >= self.GROUPED_TC_PAIRS and self._routed_tcgen05(ctx, h, w_gate_up, w_down, ids, weights,
+                                                                                x, kind, limit, alpha, scale_input, gated):
             return
-        if packed:
+        if grouped:
             # on the tensor cores: pairs sorted by expert on the device, two grouped products, a weighted sum
             self._on_device(h, w_gate_up, w_down, ids, weights, x)
             _need(h.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous() and ids.is_contiguous()
                   and weights.is_contiguous() and x.is_contiguous() and x.dtype == torch.float32
-                  and tuple(w_gate_up.shape) == (E, 128 * ((F + 63) // 64), K) and x.shape == (T, N) and ids.dtype == torch.int32
+                  and tuple(w_gate_up.shape) == (E, 128 * ((F + 63) // 64) if gated else F, K) and x.shape == (T, N) and ids.dtype == torch.int32
                   and weights.dtype == torch.float32 and w_gate_up.dtype == w_down.dtype == torch.bfloat16,
                   "routed_feed_forward: shapes")
             L = self.mixers
@@ -761,20 +818,27 @@ class CudaOps:
             y = ctx.ws.get("expert_rows", (T * top, N), torch.float32)
             self._check(L, L.gb_moe_grouped(
                 h.data_ptr(), w_gate_up.data_ptr(), w_down.data_ptr(), ids.data_ptr(), weights.data_ptr(), x.data_ptr(),
-                T, top, E, F, K, N, self.GATE_ACTS[kind], float(limit), float(alpha), 1, int(scale_input), index.data_ptr(),
+                T, top, E, F, K, N, self.GATE_ACTS[kind] if gated else self.UNARY_ACTS[kind], float(limit), float(alpha),
+                1 if gated else 2, int(scale_input), index.data_ptr(),
                 act.data_ptr(), y.data_ptr(), self._stream()), "moe_grouped", 4)
             return
         act = ctx.ws.get("expert_act", (T, top, F), h.dtype)
-        self.moe_gate_up(h, w_gate_up, ids, act, kind, limit, weights if scale_input else None)
+        if gated:
+            self.moe_gate_up(h, w_gate_up, ids, act, kind, limit, weights if scale_input else None)
+        else:
+            self.moe_up(h, w_gate_up, ids, act, kind, weights if scale_input else None)
         self.moe_down(act, w_down, ids, None if scale_input else weights, x, alpha)
 
-    def _routed_tcgen05(self, ctx, h, w_gate_up, w_down, ids, weights, x, kind, limit, alpha, scale_input=False) -> bool:
+    def _routed_tcgen05(self, ctx, h, w_gate_up, w_down, ids, weights, x, kind, limit, alpha, scale_input=False,
+                        gated=True) -> bool:
         """Many pairs: sorted by expert into blocks of 128 rows (padding rows zero), then the two
         products on the tcgen05 many-token kernel with each block's expert read from a list."""
         T, top = ids.shape
         E, N, F = w_down.shape
         K = h.shape[1]
         L, tc = self.mixers, self.tc
+        if not gated and kind not in tc.STORE_ACTS:
+            return False
         rows = int(L.gb_moe_padded_rows(T * top, E))
         blocks = rows // 128
         gu_rows = w_gate_up.shape[1]
@@ -795,7 +859,10 @@ class CudaOps:
                                                self._stream()), "moe_padded_prepare", 2)
         block_gu = index.data_ptr() + 4 * T * top
         block_dn = block_gu + 4 * blocks
-        tc.grouped(a, w_gate_up, act, F, E, block_gu, 2, gate_act=self.GATE_ACTS[kind], gate_limit=limit)
+        if gated:
+            tc.grouped(a, w_gate_up, act, F, E, block_gu, 2, gate_act=self.GATE_ACTS[kind], gate_limit=limit)
+        else:
+            tc.grouped(a, w_gate_up, act, F, E, block_gu, 0, gate_act=tc.STORE_ACTS[kind])
         tc.grouped(act, w_down, y, N, E, block_dn, 0)
         self._check(L, L.gb_moe_combine(y.data_ptr(), index.data_ptr(), None if scale_input else weights.data_ptr(), x.data_ptr(), T, top, N,
                                         float(alpha), self._stream()), "moe_combine")
@@ -1055,22 +1122,24 @@ class CudaOps:
 
     # ------------------------------------------------------------------ normed queries and keys; sublayers normed behind
     def qk_norm_rope_append(self, src, cols, q_out, k_pool, v_pool, positions, token_req, block_table, heads, kv_heads,
-                            dim, vdim, q_weight, k_weight, eps, rotary, page_size):
+                            dim, vdim, q_weight, k_weight, eps, rotary, page_size, query_growth=None):
         """From a projected 32-bit row ``src [T, P]`` with ``cols = (q, k, v)`` the first columns of
         queries (``heads dim``), keys (``kv_heads dim``) and values (``kv_heads vdim``; the keys' own
         columns where the values are the keys as projected): queries and keys are divided by their root
         mean square per head (``q_weight [heads, dim]``, ``k_weight [dim]``, 32-bit; None: no norm),
         then rotated (``rotary``: a ``RotaryParams`` over ``dim``, or None); queries go to ``q_out
-        [T, heads, dim]``, keys and the untouched values into their pages."""
+        [T, heads, dim]``, keys and the untouched values into their pages. ``query_growth = (coef, every)``: the
+        query at position ``p`` is multiplied by ``1 + coef ln(floor((p + 1) / every) + 1)``. ``kv_heads`` 0: queries
+        only, the pools are not touched."""
         self._on_device(src, q_out, k_pool, v_pool, positions, token_req, block_table, q_weight, k_weight)
         T = src.shape[0]
         cq, ck, cv = (int(c) for c in cols)
         _need(src.dtype == torch.float32 and src.stride(1) == 1, "qk_norm_rope_append: a float32 row")
         _need(max(cq + heads * dim, ck + kv_heads * dim, cv + kv_heads * vdim) <= src.shape[1], "qk_norm_rope_append: columns")
         _need(q_out.is_contiguous() and tuple(q_out.shape) == (T, heads, dim), "qk_norm_rope_append: q_out shape")
-        _need(k_pool.dtype == q_out.dtype == v_pool.dtype and k_pool.is_contiguous() and v_pool.is_contiguous()
+        _need(kv_heads == 0 or (k_pool.dtype == q_out.dtype == v_pool.dtype and k_pool.is_contiguous() and v_pool.is_contiguous()
               and tuple(k_pool.shape[1:]) == (kv_heads, page_size, dim)
-              and tuple(v_pool.shape[1:]) == (kv_heads, page_size, vdim), "qk_norm_rope_append: pool shapes")
+              and tuple(v_pool.shape[1:]) == (kv_heads, page_size, vdim)), "qk_norm_rope_append: pool shapes")
         _need(block_table.dtype == torch.int32 and block_table.is_contiguous() and positions.dtype == torch.int32
               and token_req.dtype == torch.int32, "qk_norm_rope_append: int32 indices")
         _need(q_weight is None or (q_weight.dtype == torch.float32 and q_weight.is_contiguous()
@@ -1081,14 +1150,15 @@ class CudaOps:
         if rotary is not None:
             _need(rotary.head_dim == dim, "qk_norm_rope_append: rotary is for another head width")
             inv, inter = self.inv_freq(rotary), int(rotary.interleaved)
+        coef, every = query_growth if query_growth is not None else (0.0, 0)
         L = self.state_lib
         self._check(L, L.gb_qk_norm_rope_append(
             src.data_ptr(), src.stride(0), cq, ck, cv, q_out.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
             _tag(q_out, "q_out"), positions.data_ptr(), token_req.data_ptr(), block_table.data_ptr(), block_table.shape[1],
             T, heads, kv_heads, dim, vdim, _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(inv), inter, page_size,
-            self._stream()), "qk_norm_rope_append")
+            float(coef), int(every), self._stream()), "qk_norm_rope_append")
 
-    UNARY_ACTS = {"sigmoid": 0, "silu": 1, "relu2": 2, "tanh": 3}
+    UNARY_ACTS = {"sigmoid": 0, "silu": 1, "relu2": 2, "tanh": 3, "gelu": 4}
 
     def gate_mul(self, x, gate, kind: str = "sigmoid"):
         """``x <- x * act(gate)`` in place; ``gate [T, n]`` 32-bit logits (a column range of a wider
@@ -1104,7 +1174,7 @@ class CudaOps:
 
     def activation(self, z, out, kind: str):
         """``out = act(z)`` elementwise, 32-bit arithmetic; ``act`` = ``relu2`` (the square of
-        relu), ``tanh``, ``sigmoid`` or ``silu``. Both may be column ranges of wider rows."""
+        relu), ``tanh``, ``sigmoid``, ``silu`` or ``gelu`` (the exact one). Both may be column ranges of wider rows."""
         self._on_device(z, out)
         T, n = z.shape
         _need(tuple(out.shape) == (T, n) and z.stride(1) == 1 and out.stride(1) == 1, "activation: shapes")
@@ -1247,6 +1317,58 @@ class CudaOps:
         self._check(L, L.gb_mingru(proj.data_ptr(), proj.stride(0), cz, cu, cg, _ptr(bias_z), _ptr(bias_u), b.cu_q.data_ptr(),
                                    b.slots.data_ptr(), state.data_ptr(), state.stride(0), out.data_ptr(), _tag(out, "mingru out"),
                                    R, W, int(b.max_q_len), _ptr(scratch), self._stream()), "mingru", 2 if need else 1)
+
+    # ------------------------------------------------------------------ a state space with one decay per head and token
+    #: tokens of a step's longest request from which the recurrence runs in chunks on the tensor cores
+    SSD_CHUNK_TOKENS = 24
+
+    def state_space(self, ctx, proj, cols, conv_w, conv_b, rate, dt_bias, skip, norm_w, norm_groups, eps, state, heads,
+                    groups, dim, vdim, out):
+        """The recurrent part of a state-space mixer for one step. ``proj [T, P]`` (32-bit): the projected
+        row; ``cols = (z, x, d)``: the first columns of the gate (``H vdim``), of the convolved channels (x
+        of all heads, then ``B`` and ``C`` of all groups, ``dim`` each) and of the step sizes (``H``). ``conv_w [C,
+        taps]``, ``conv_b [C]`` or None; ``rate, dt_bias, skip [H]``; ``norm_w [H vdim]`` (all 32-bit). Per head:
+        ``dt = softplus(d + dt_bias)``, ``S <- exp(-rate dt) S + x (dt B)^T``, ``y = S C + skip x``; then ``out = v /
+        rms(v) * norm_w`` with ``v = y silu(z)``, the mean over each of ``norm_groups`` equal parts. The convolved
+        activations are rounded to ``out``'s dtype. ``state [slots, H vdim dim + (taps - 1) C]`` (32-bit: ``S [H, vdim,
+        dim]``, then the kept last inputs of the convolution) is advanced for the batch's requests."""
+        b = ctx.batch
+        self._on_device(proj, conv_w, conv_b, rate, dt_bias, skip, norm_w, state, out)
+        T, H, G = proj.shape[0], int(heads), int(groups)
+        cz, cx, cd = (int(c) for c in cols)
+        inner, taps = H * vdim, conv_w.shape[1]
+        C, n_state = inner + 2 * G * dim, inner * dim
+        _need(proj.dtype == torch.float32 and proj.stride(1) == 1 and max(cz + inner, cx + C, cd + H) <= proj.shape[1],
+              "state_space: a float32 row with three column ranges")
+        _need(all(v is None or (v.dtype == torch.float32 and v.is_contiguous()) for v in (conv_w, conv_b, rate, dt_bias, skip, norm_w))
+              and conv_w.shape[0] == C and (conv_b is None or conv_b.numel() == C) and rate.numel() == dt_bias.numel() == skip.numel() == H
+              and norm_w.numel() == inner and inner % norm_groups == 0, "state_space: weights")
+        _need(state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] == n_state + (taps - 1) * C, "state_space: state")
+        _need(out.is_contiguous() and tuple(out.shape) == (T, inner), "state_space: out")
+        L, P, stride = self.ssd_lib, proj.stride(0), state.shape[1]
+        kept = state.data_ptr() + 4 * n_state
+        y = ctx.ws.get("ssd_y", (T, inner), torch.float32)
+        tag = _tag(out, "state_space out")
+        if b.max_q_len == 1:
+            self._check(L, L.gb_ssd_decode(
+                proj.data_ptr(), P, cx, cd, conv_w.data_ptr(), _ptr(conv_b), taps, kept, stride, rate.data_ptr(), dt_bias.data_ptr(),
+                skip.data_ptr(), b.slots.data_ptr(), state.data_ptr(), stride, T, H, G, dim, vdim, tag, y.data_ptr(), self._stream()),
+                "ssd_decode")
+        else:
+            act = ctx.ws.get("ssd_act", (T, C), out.dtype)
+            step = ctx.ws.get("ssd_step", (T, 2 * H), torch.float32)
+            self._check(L, L.gb_ssd_prepare(
+                proj.data_ptr(), P, cx, cd, conv_w.data_ptr(), _ptr(conv_b), taps, kept, stride, rate.data_ptr(), dt_bias.data_ptr(),
+                b.token_req.data_ptr(), b.cu_q.data_ptr(), b.slots.data_ptr(), act.data_ptr(), tag, step.data_ptr(), T, H, G, dim,
+                vdim, self._stream()), "ssd_prepare")
+            if not (b.max_q_len >= self.SSD_CHUNK_TOKENS and self.tc is not None and self.tc.ssd_chunk(
+                    act, step, skip, b.cu_q, b.slots, state, b.num_requests, H, G, dim, vdim, y)):
+                self._check(L, L.gb_ssd_recurrence(
+                    act.data_ptr(), tag, step.data_ptr(), skip.data_ptr(), b.cu_q.data_ptr(), b.slots.data_ptr(), state.data_ptr(),
+                    stride, b.num_requests, H, G, dim, vdim, y.data_ptr(), self._stream()), "ssd_recurrence")
+        self._check(L, L.gb_ssd_finish(
+            y.data_ptr(), proj.data_ptr(), P, cz, cx, norm_w.data_ptr(), float(eps), out.data_ptr(), tag, T, int(norm_groups), inner,
+            kept, stride, b.cu_q.data_ptr(), b.slots.data_ptr(), b.num_requests, C, taps, self._stream()), "ssd_finish")
 
     # ------------------------------------------------------------------ a short convolution in front of attention
     def conv_qkv_append(self, ctx, proj, bias, conv_w, taps, state, q_out, k_pool, v_pool, block_table, heads, kv_heads,

@@ -11,7 +11,8 @@ from ctypes import c_void_p, c_int, c_float
 
 import torch
 
-from ..csrc.build import load_kernel_lib, attention_lib_name, latent_attention_lib_name, capped_attention_lib_name
+from ..csrc.build import (load_kernel_lib, attention_lib_name, latent_attention_lib_name, capped_attention_lib_name,
+                          ssd_lib_name)
 
 _WAIT_NAMES = {1: "an operand tile never arrived (TMA)", 2: "a pipeline stage was never released",
                3: "the accumulator never completed", 4: "copies in flight did not land while winding down",
@@ -56,6 +57,7 @@ class TensorCoreKernels:
         self._attn = {}
         self._latent = {}
         self._capped = {}
+        self._ssd = {}
         # The weights that the products of a step stream, in launch order: recorded during one run
         # (``record_streams``) and replayed as hints during the next (``hint_streams``), so that every
         # few-token product asks for the weights of the product behind it to be brought into L2 while
@@ -136,7 +138,8 @@ class TensorCoreKernels:
     def grouped(self, a, w, out, n_out, groups, block_w_row, epi, gate_act: int = 0, gate_limit: float = 0.0) -> None:
         """A grouped product: ``a [rows, K]`` sorted by group in blocks of 128 rows, ``w [groups, *, K]``
         the groups' weights, ``block_w_row``: device address of the int32 list that gives every block
-        the first weight row of its group. ``epi`` 0: ``out = a w^T``; 2: the gated epilogue."""
+        the first weight row of its group. ``epi`` 0: ``out = a w^T`` (or, with ``gate_act`` one of
+        ``STORE_ACTS``, that activation of it); 2: the gated epilogue."""
         rows, K = a.shape
         self._stream(w)
         code = self.lib.gb_gemm_tc_grouped(a.data_ptr(), w.data_ptr(), out.data_ptr(), rows, int(n_out), K, int(groups),
@@ -156,10 +159,10 @@ class TensorCoreKernels:
                             sums_out=emit.sums.data_ptr(), sums_ld=emit.sums.shape[1])
         return self._gemm(a, w, out, w.shape[0], 1 if accumulate else 0, fold, alpha=alpha)
 
-    STORE_ACTS = {"relu2": 3, "tanh": 4}
+    STORE_ACTS = {"relu2": 3, "tanh": 4, "gelu": 6}
 
     def linear_act(self, a, w, out, kind: str) -> bool:
-        """``out = act(a w^T)`` in bfloat16, the activation (``relu2``, ``tanh``) on the 32-bit sums in
+        """``out = act(a w^T)`` in bfloat16, the activation (``relu2``, ``tanh``, ``gelu``) on the 32-bit sums in
         the product's epilogue."""
         if w.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or kind not in self.STORE_ACTS:
             return False
@@ -410,4 +413,28 @@ class TensorCoreKernels:
             int(splits), None if scratch is None else scratch.data_ptr(), need,
             None if sink_values is None else sink_values.data_ptr(), self.ops._stream())
         self.ops._check(lib, code, "latent_attention", 1 if splits == 1 else 2)
+        return True
+
+    # ------------------------------------------------------------------ a state space over long stretches of tokens
+    @staticmethod
+    def takes_ssd(state_dim: int, head_dim: int) -> bool:
+        """Sizes the kernel is compiled for: whole blocks of 16 of both, states that fit a CTA's registers."""
+        return state_dim % 16 == 0 and head_dim % 16 == 0 and 16 <= state_dim <= 256 and head_dim >= 16
+
+    def ssd_chunk(self, act, step, skip, cu_q, slots, state, num_requests, heads, groups, state_dim, head_dim, y) -> bool:
+        """The recurrence of ``CudaOps.state_space`` from its prepared rows, chunk by chunk on the tensor
+        cores; False where the kernel does not take the sizes."""
+        if act.dtype != torch.bfloat16 or not self.takes_ssd(state_dim, head_dim):
+            return False
+        lib = self._ssd.get((state_dim, head_dim))
+        if lib is None:
+            lib = load_kernel_lib(ssd_lib_name(state_dim, head_dim))
+            lib.gb_last_error.restype = ctypes.c_char_p
+            lib.gb_ssd_chunk.argtypes = [c_void_p] * 6 + [ctypes.c_longlong] + [c_int] * 3 + [c_void_p, c_void_p]
+            lib.gb_ssd_chunk.restype = c_int
+            self._ssd[(state_dim, head_dim)] = lib
+        code = lib.gb_ssd_chunk(act.data_ptr(), step.data_ptr(), skip.data_ptr(), cu_q.data_ptr(), slots.data_ptr(),
+                                state.data_ptr(), state.stride(0), int(num_requests), int(heads), int(groups), y.data_ptr(),
+                                self.ops._stream())
+        self.ops._check(lib, code, "ssd_chunk")
         return True

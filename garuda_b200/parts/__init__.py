@@ -5,15 +5,16 @@ from .base import (Part, Norm, PositionEncoding, Mixer, FeedForward, ResidualBra
                    register_feed_forward, register_norm, register_position_encoding,
                    register_block, register_branch, register_connection, register_gate,
                    SublayerGate)
-from .norm import RMSNorm, LayerNorm
+from .norm import RMSNorm, LayerNorm, DynamicTanh
 from .rotary import Rotary, NoPositions, RotaryParams
 from .attention import PagedAttention, CappedSinkAttention, NormedKeyAttention, ConvolvedAttention
 from .mingru import MinGRU
+from .state_space import StateSpaceDuality
 from .delta_rule import ChannelDeltaRule, HeadDeltaRule, GeneralDeltaRule
 from .mlp import SwiGLU, GatedFeedForward, PlainFeedForward
 from .latent_attention import LatentAttention
 from .experts import RoutedExperts
 from .token_side import TokenSide
-from .block import BlockSpec, PreNormBlock, SublayerNormBlock, PostNormBlock, LinearSigmoidGate, BranchOutputs
+from .block import BlockSpec, PreNormBlock, SublayerNormBlock, PostNormBlock, ParallelBlock, LinearSigmoidGate, BranchOutputs
 from .parallel import ParallelMixers
 from .hyper import StreamMixing, StreamPreNormBlock

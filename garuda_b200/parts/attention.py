@@ -209,14 +209,22 @@ class NormedKeyAttention(Mixer):
 
     The temperature multiplies the query's norm weight when the weights are loaded (the rotation
     is linear), so the attention kernel sees one scale. One product makes ``[q | k | (v) | gate]``
-    in 32-bit; one kernel norms, rotates and stores. ``names``: the tensors' local names."""
+    in 32-bit; one kernel norms, rotates and stores. ``names``: the tensors' local names.
+
+    Further options, off unless given: ``qk_norm_weight=False``: the norms have no weight; ``query_growth =
+    (coef, every)``: the query at position ``p`` is multiplied by ``1 + coef ln(floor((p + 1) / every) + 1)``;
+    ``sink``: ``exp(sink_n)``, a learned number per head, joins the softmax's denominator (no key, no value,
+    not scaled); ``reads_shared_cache``: the layer has queries only and reads the keys, as they are
+    cached, and values of the call that its entry of the run order names."""
     graph_safe = True
+    scales_residual = True
 
     def __init__(self, width: int, heads: int, kv_heads: int, dim: int, scale: Optional[float] = None,
                  window: Optional[int] = None, rot_base: Optional[float] = None, rot_dims: int = 0,
                  rot_layout: str = "interleaved", qk_norm: bool = True, eps: float = 1e-6, temperature: bool = True,
                  values: str = "keys", vdim: Optional[int] = None, gate: bool = True, names: Optional[dict] = None,
-                 init_std: float = 0.02):
+                 init_std: float = 0.02, qk_norm_weight: bool = True, sink: bool = False, query_growth=None,
+                 reads_shared_cache: bool = False):
         if heads % kv_heads:
             raise ValueError(f"{heads} query heads are not a multiple of {kv_heads} kv heads")
         if values not in ("keys", "projected"):
@@ -229,8 +237,15 @@ class NormedKeyAttention(Mixer):
         self.window = int(window) if window else None
         self.qk_norm, self.eps, self.temperature = bool(qk_norm), float(eps), bool(temperature)
         self.values, self.gate = values, bool(gate)
+        self.qk_norm_weight, self.sink, self.reads_shared_cache = bool(qk_norm_weight), bool(sink), bool(reads_shared_cache)
+        self.query_growth = None
+        if query_growth is not None:
+            coef, every = query_growth
+            if int(every) < 1:
+                raise ValueError(f"queries grow every {every} positions")
+            self.query_growth = (float(coef), int(every))
         self.names = dict({"q": "q", "k": "k", "v": "v", "g": "g", "o": "o", "q_norm": "q.norm", "k_norm": "k.norm",
-                           "temp": "temp"}, **(names or {}))
+                           "temp": "temp", "sink": "sink"}, **(names or {}))
         self.init_std = float(init_std)
         self.rotary = None
         if rot_base is not None and rot_dims:
@@ -245,15 +260,19 @@ class NormedKeyAttention(Mixer):
 
     def tensors(self):
         init, n = ("normal", self.init_std), self.names
-        t = {n["q"]: TensorSpec((self.q_dim, self.width), init=init), n["k"]: TensorSpec((self.k_dim, self.width), init=init),
-             n["o"]: TensorSpec((self.width, self.ctx_dim), init=init)}
-        if self.values == "projected":
+        t = {n["q"]: TensorSpec((self.q_dim, self.width), init=init), n["o"]: TensorSpec((self.width, self.ctx_dim), init=init)}
+        if not self.reads_shared_cache:
+            t[n["k"]] = TensorSpec((self.k_dim, self.width), init=init)
+        if self.values == "projected" and not self.reads_shared_cache:
             t[n["v"]] = TensorSpec((self.v_dim, self.width), init=init)
         if self.gate:
             t[n["g"]] = TensorSpec((self.ctx_dim, self.width), init=init)
-        if self.qk_norm:
+        if self.qk_norm and self.qk_norm_weight:
             t[n["q_norm"]] = TensorSpec((self.dim,), role="vector", init=("normal_about_one", 0.1))
-            t[n["k_norm"]] = TensorSpec((self.dim,), role="vector", init=("normal_about_one", 0.1))
+            if not self.reads_shared_cache:
+                t[n["k_norm"]] = TensorSpec((self.dim,), role="vector", init=("normal_about_one", 0.1))
+        if self.sink:
+            t[n["sink"]] = TensorSpec((self.heads,), role="vector", init=("normal", 1.0))
         if self.temperature:
             t[n["temp"]] = TensorSpec((self.heads,), role="vector", init=("normal_about_one", 0.2))
         return t
@@ -264,43 +283,54 @@ class NormedKeyAttention(Mixer):
     def load(self, tensors, ops, dtype):
         super().load(tensors, ops, dtype)
         n = self.names
-        rows = [tensors[n["q"]], tensors[n["k"]]]
-        self.col_q, self.col_k = 0, self.q_dim
-        self.col_v = self.col_k
-        at = self.q_dim + self.k_dim
-        if self.values == "projected":
-            rows.append(tensors[n["v"]])
-            self.col_v, at = at, at + self.v_dim
+        rows = [tensors[n["q"]]]
+        self.col_q = self.col_k = self.col_v = 0
+        at = self.q_dim
+        if not self.reads_shared_cache:
+            rows.append(tensors[n["k"]])
+            self.col_k = self.col_v = at
+            at += self.k_dim
+            if self.values == "projected":
+                rows.append(tensors[n["v"]])
+                self.col_v, at = at, at + self.v_dim
         self.col_g = at
         if self.gate:
             rows.append(tensors[n["g"]])
         self.w_in = torch.cat(rows, dim=0).contiguous()
         self.w_o = tensors[n["o"]].contiguous()
-        self.k_weight = tensors[n["k_norm"]].float().contiguous() if self.qk_norm else None
-        self.q_weight = None
+        self.sinks = tensors[n["sink"]].float().contiguous() if self.sink else None
+        self.q_weight = self.k_weight = None
         if self.qk_norm:
-            per_head = tensors[n["q_norm"]].float()[None, :].expand(self.heads, self.dim)
+            ones = torch.ones(self.dim, dtype=torch.float32, device=self.w_in.device)
+            if not self.reads_shared_cache:
+                self.k_weight = tensors[n["k_norm"]].float().contiguous() if self.qk_norm_weight else ones
+            per_head = tensors[n["q_norm"]].float() if self.qk_norm_weight else ones
+            per_head = per_head[None, :].expand(self.heads, self.dim)
             if self.temperature:
                 per_head = per_head * tensors[n["temp"]].float()[:, None]
             self.q_weight = per_head.contiguous()
 
-    def forward(self, ctx, h, cache, residual=None, out_name: str = "attn_y"):
+    def forward(self, ctx, h, cache, residual=None, out_name: str = "attn_y", alpha: float = 1.0):
         b, ops, ws = ctx.batch, self.ops, ctx.ws
         T = h.shape[0]
+        if cache.writes == self.reads_shared_cache:
+            raise ValueError("the run order and the layer disagree about whose keys and values are read")
         proj = ws.get("attn_proj", (T, self.w_in.shape[0]), torch.float32)
         ops.linear(h, self.w_in, proj)
         q = ws.get("q_heads", (T, self.heads, self.dim), self.dtype)
+        kw = {} if self.query_growth is None else {"query_growth": self.query_growth}
         ops.qk_norm_rope_append(proj, (self.col_q, self.col_k, self.col_v), q, cache.k, cache.v, b.positions, b.token_req,
-                                cache.block_table, self.heads, self.kv_heads, self.dim, self.vdim, self.q_weight,
-                                self.k_weight, self.eps, self.rotary, cache.page_size)
+                                cache.block_table, self.heads, 0 if self.reads_shared_cache else self.kv_heads, self.dim,
+                                self.vdim, self.q_weight, self.k_weight, self.eps, self.rotary, cache.page_size, **kw)
         out = ws.get("attn_ctx", (T, self.ctx_dim), self.dtype)
+        kw = {} if self.sinks is None else {"sink_values": self.sinks}
         ops.paged_attention(q, cache.k, cache.v, cache.block_table, b.cu_q, b.kv_lens, b.token_req, out,
                             self.scale, self.window or 0, cache.page_size, b.num_requests, b.max_q_len, b.max_kv_len,
-                            ws=ws, min_q_len=b.min_q_len)
+                            ws=ws, min_q_len=b.min_q_len, **kw)
         if self.gate:
             ops.gate_mul(out, proj[:, self.col_g:self.col_g + self.ctx_dim], "sigmoid")
         if residual is not None:
-            ops.linear(out, self.w_o, residual, accumulate=True)
+            ops.linear(out, self.w_o, residual, accumulate=True, alpha=alpha)
             return None
         y = ws.get(out_name, (T, self.width), torch.float32)
         ops.linear(out, self.w_o, y)

@@ -382,3 +382,48 @@ class PostNormBlock:
 
 
 _NO_CACHE = object()
+
+
+@register_block("parallel")
+class ParallelBlock:
+    """A layer with one norm whose output both sublayers read: ``x <- x + m * (mixer(h) + ffn(h))`` with ``h =
+    norm(x)`` (``BlockSpec.mixer_norm``) and ``m = BlockSpec.residual_mult``. The residual is 32-bit; each
+    sublayer adds into it (in its last product's epilogue, where it can): ``h`` has been taken by then, so
+    the two sums may follow one another."""
+
+    def __init__(self, spec: BlockSpec):
+        if spec.feed_forward_norm is not None or spec.branches or spec.mixer_connection is not None or spec.mixer_gate is not None:
+            raise ValueError("a layer whose sublayers share their input has one norm and takes no branches, streams or gates")
+        self.spec = spec
+        self.mixer = build_part("mixer", spec.mixer)
+        self.norm = build_part("norm", spec.mixer_norm)
+        self.feed_forward = build_part("feed_forward", spec.feed_forward) if spec.feed_forward else None
+        self.mult = float(spec.residual_mult)
+
+    def parts(self):
+        s = self.spec
+        out = [(self.norm, s.mixer_norm.prefix), (self.mixer, s.mixer.prefix)]
+        if self.feed_forward is not None:
+            out.append((self.feed_forward, s.feed_forward.prefix))
+        return out
+
+    @property
+    def graph_safe(self):
+        return all(part.graph_safe for part, _ in self.parts())
+
+    _run_scaled = PreNormBlock._run
+
+    def _run(self, ctx, part, x, h, *cache):
+        if self.mult != 1.0:
+            return self._run_scaled(ctx, part, x, h, *cache)
+        y = part.forward(ctx, h, *cache, residual=x)
+        if y is not None:
+            ctx.ops.residual_add(x, y)
+
+    def forward(self, ctx, x, cache):
+        ctx.pending_norm = None
+        h = self.norm.forward(ctx, x)
+        self._run(ctx, self.mixer, x, h, cache)
+        if self.feed_forward is not None:
+            self._run(ctx, self.feed_forward, x, h)
+        return None

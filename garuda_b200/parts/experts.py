@@ -13,9 +13,10 @@ Variants, by constructor parameter: ``router_score="sigmoid"`` weighs a chosen e
 (not renormalized over the chosen either);
 ``scale_input=True`` puts the weight on what goes into the expert, ``out = sum_chosen
 expert_e(weight_e * h)``; ``router_bias=False`` drops ``b_r``; ``activation="silu"`` is the plain
-SiLU gate.
+SiLU gate; ``gated=False`` makes an expert ``W_down act(W_up h)`` without a gate (``activation`` = ``"gelu"``,
+the exact one, or any activation of ``PlainFeedForward`` without numbers of its own).
 
-Tensor names: ``router``, ``router.b``, ``e<i>.gate|up|down``, ``shared.gate|up|down``.
+Tensor names: ``router``, ``router.b``, ``e<i>.gate|up|down`` (no ``gate`` without one), ``shared.gate|up|down``.
 """
 from __future__ import annotations
 
@@ -24,6 +25,9 @@ from typing import Optional
 import torch
 
 from .base import FeedForward, TensorSpec, register_feed_forward
+
+#: activations of one value that the expert and the plain feed-forward kernels know
+PLAIN_ACTIVATIONS = ("relu2", "silu", "tanh", "sigmoid", "gelu")
 
 
 @register_feed_forward("routed_experts")
@@ -34,7 +38,10 @@ class RoutedExperts(FeedForward):
     def __init__(self, width: int, experts: int, top: int, inner: int, activation: str = "clamped_swish",
                  limit: float = 0.0, shared_inner: Optional[int] = None, shared_limit: float = 0.0,
                  router_bias: bool = True, init_std: float = 0.02, router_score: str = "softmax_chosen",
-                 scale_input: bool = False):
+                 scale_input: bool = False, gated: bool = True):
+        if not gated and (shared_inner or activation not in PLAIN_ACTIVATIONS):
+            raise ValueError(f"experts without a gate take {PLAIN_ACTIVATIONS} and no shared expert, got {activation!r}")
+        self.gated = bool(gated)
         if router_score not in ("softmax_chosen", "sigmoid", "softmax_all"):
             raise ValueError(f"unknown router score {router_score!r}")
         self.router_score, self.scale_input = router_score, bool(scale_input)
@@ -53,7 +60,8 @@ class RoutedExperts(FeedForward):
         if self.router_bias:
             t["router.b"] = TensorSpec((self.experts,), role="vector", init=("normal", 0.02))
         for e in range(self.experts):
-            t[f"e{e}.gate"] = TensorSpec((self.inner, self.width), init=init)
+            if self.gated:
+                t[f"e{e}.gate"] = TensorSpec((self.inner, self.width), init=init)
             t[f"e{e}.up"] = TensorSpec((self.inner, self.width), init=init)
             t[f"e{e}.down"] = TensorSpec((self.width, self.inner), init=init)
         if self.shared_inner:
@@ -67,9 +75,12 @@ class RoutedExperts(FeedForward):
         self.w_router = tensors["router"].contiguous()
         self.b_router = tensors["router.b"].float().contiguous() if self.router_bias else None
         E = self.experts
-        # the experts' gate and up rows stacked in the kernels' layout; [E, width, inner]
-        self.w_gate_up = ops.pack_expert_gate_up([tensors[f"e{e}.gate"] for e in range(E)],
-                                                 [tensors[f"e{e}.up"] for e in range(E)])
+        # the experts' gate and up rows stacked in the kernels' layout, or the up rows alone; [E, width, inner]
+        if self.gated:
+            self.w_gate_up = ops.pack_expert_gate_up([tensors[f"e{e}.gate"] for e in range(E)],
+                                                     [tensors[f"e{e}.up"] for e in range(E)])
+        else:
+            self.w_gate_up = torch.stack([tensors[f"e{e}.up"] for e in range(E)]).contiguous()
         self.w_down = torch.stack([tensors[f"e{e}.down"] for e in range(E)]).contiguous()
         if self.shared_inner:
             self.w_shared_gate_up = ops.pack_gate_up(tensors["shared.gate"], tensors["shared.up"])
@@ -85,14 +96,15 @@ class RoutedExperts(FeedForward):
             alpha = 1.0
         ids = ws.get("expert_ids", (T, self.top), torch.int32)
         weights = ws.get("expert_weights", (T, self.top), torch.float32)
-        if self.router_score == "softmax_chosen" and not self.scale_input:
+        if self.router_score == "softmax_chosen" and not self.scale_input and self.gated:
             ops.route_topk(h, self.w_router, self.b_router, self.top, ids, weights)
             ops.routed_feed_forward(ctx, h, self.w_gate_up, self.w_down, ids, weights, target, self.activation,
                                     self.limit, alpha)
         else:
             ops.route_topk(h, self.w_router, self.b_router, self.top, ids, weights, score=self.router_score)
+            kw = {} if self.gated else {"gated": False}
             ops.routed_feed_forward(ctx, h, self.w_gate_up, self.w_down, ids, weights, target, self.activation,
-                                    self.limit, alpha, scale_input=self.scale_input)
+                                    self.limit, alpha, scale_input=self.scale_input, **kw)
         if self.shared_inner:
             act = ws.get("shared_act", (T, self.shared_inner), self.dtype)
             ops.linear_gated(ctx, h, self.w_shared_gate_up, act, self.activation, self.shared_limit)

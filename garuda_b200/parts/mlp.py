@@ -99,7 +99,7 @@ class GatedFeedForward(FeedForward):
 @register_feed_forward("plain")
 class PlainFeedForward(FeedForward):
     """``down(act(up h))`` without a gate: ``activation`` is ``"relu2"`` (the square of relu),
-    ``"silu"``, ``"tanh"``, ``"sigmoid"`` or ``"xielu"``, computed in 32-bit on the product's 32-bit
+    ``"silu"``, ``"tanh"``, ``"sigmoid"``, ``"gelu"`` (the exact one) or ``"xielu"``, computed in 32-bit on the product's 32-bit
     result and rounded once. ``names``: the tensors' local names.
 
     ``xielu`` has two learned numbers ``p, q`` (tensor ``act_name``, ``[2]``): ``softplus(p) z^2 + z / 2``
@@ -111,7 +111,7 @@ class PlainFeedForward(FeedForward):
 
     def __init__(self, width: int, inner: int, activation: str = "relu2", names=("up", "down"), init_std: float = 0.02,
                  act_name: str = "act"):
-        if activation not in ("relu2", "silu", "tanh", "sigmoid", "xielu"):
+        if activation not in ("relu2", "silu", "tanh", "sigmoid", "gelu", "xielu"):
             raise ValueError(f"unknown activation {activation!r}")
         self.width, self.inner, self.activation = int(width), int(inner), activation
         self.names = tuple(names)

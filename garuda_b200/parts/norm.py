@@ -1,5 +1,6 @@
 """RMS norm: ``x * 1/sqrt(mean(x^2) + eps) * weight``, and layer norm:
-``(x - mean) / sqrt(var + eps) * weight + bias``.
+``(x - mean) / sqrt(var + eps) * weight + bias``; and a norm without statistics,
+``tanh(alpha * x) * weight + bias``.
 
 garuda/src/simd/mod.rs:166-173 (eps inside the root, added to the mean) and
 garuda/src/llama/mod.rs:733-738 (scale, then a plain multiply by the weight).
@@ -94,4 +95,34 @@ class LayerNorm(Norm):
         n = x.shape[0] if rows is None else rows.shape[0]
         out = ctx.ws.get(out_name, (n, self.width), self.dtype)
         self.ops.layernorm(x, self.weight, self.bias, self.eps, out, rows)
+        return out
+
+
+@register_norm("dynamic_tanh")
+class DynamicTanh(Norm):
+    """``tanh(alpha * x) * weight + bias`` per channel with a learned number ``alpha``: no mean, no variance.
+    32-bit in the kernel, the result rounded to the compute dtype. ``weight_name``: the weight's local
+    name; the other two tensors are that name with ``.alpha`` and ``.b`` added."""
+    graph_safe = True
+
+    def __init__(self, width: int, weight_name: str = "weight"):
+        self.width, self.weight_name = int(width), weight_name
+
+    def tensors(self):
+        n = self.weight_name
+        return {n: TensorSpec((self.width,), role="vector", init=("normal_about_one", 0.1)),
+                n + ".b": TensorSpec((self.width,), role="vector", init=("normal", 0.05)),
+                n + ".alpha": TensorSpec((), role="vector", init=("uniform", 0.3, 0.9))}
+
+    def load(self, tensors, ops, dtype):
+        super().load(tensors, ops, dtype)
+        n = self.weight_name
+        self.weight, self.bias = tensors[n].float().contiguous(), tensors[n + ".b"].float().contiguous()
+        self.alpha = float(tensors[n + ".alpha"].float().reshape(-1)[0])
+
+    def forward(self, ctx, x: torch.Tensor, rows: Optional[torch.Tensor] = None,
+                out_name: str = "normed") -> torch.Tensor:
+        n = x.shape[0] if rows is None else rows.shape[0]
+        out = ctx.ws.get(out_name, (n, self.width), self.dtype)
+        self.ops.dynamic_tanh(x, self.alpha, self.weight, self.bias, out, rows)
         return out

@@ -243,13 +243,26 @@ class CpuOps:
                 total += wt * (w_down[int(ids[t, j])].float() @ act[t, j].float())
             x[t] += alpha * total
 
+    def moe_up(self, h, w_up, ids, act, kind, in_scale=None):
+        """experts without a gate: act(up_e h), w_up [E, F, K]"""
+        for t in range(h.shape[0]):
+            for j, e in enumerate(ids[t].tolist()):
+                u = w_up[e].float() @ h[t].float()
+                if in_scale is not None:
+                    u = u * in_scale[t, j]
+                act[t, j] = self._unary(u, kind).to(act.dtype)
+
     def pack_expert_gate_up(self, gates, ups):
         return torch.stack([torch.cat([g, u], 0) for g, u in zip(gates, ups)]).contiguous()
 
-    def routed_feed_forward(self, ctx, h, w_gate_up, w_down, ids, weights, x, kind, limit, alpha=1.0, scale_input=False):
+    def routed_feed_forward(self, ctx, h, w_gate_up, w_down, ids, weights, x, kind, limit, alpha=1.0, scale_input=False,
+                            gated=True):
         T, top = ids.shape
         act = torch.zeros(T, top, w_down.shape[2], dtype=h.dtype)
-        self.moe_gate_up(h, w_gate_up, ids, act, kind, limit, weights if scale_input else None)
+        if gated:
+            self.moe_gate_up(h, w_gate_up, ids, act, kind, limit, weights if scale_input else None)
+        else:
+            self.moe_up(h, w_gate_up, ids, act, kind, weights if scale_input else None)
         self.moe_down(act, w_down, ids, None if scale_input else weights, x, alpha)
 
     # ---- a norm after the sum, gates per head, xIELU, a gated recurrence per channel, convolved projections ----
@@ -406,6 +419,47 @@ class CpuOps:
             state[slot, :n_state] = S.reshape(-1)
             state[slot, n_state:] = kept.reshape(-1)
 
+    # ---- a norm without statistics; a state space with one decay per head and token ----
+    def dynamic_tanh(self, x, alpha, weight, bias, out, rows=None):
+        xs = x if rows is None else x[rows.long()]
+        out.copy_((torch.tanh(alpha * xs) * weight + bias).to(out.dtype))
+
+    def state_space(self, ctx, proj, cols, conv_w, conv_b, rate, dt_bias, skip, norm_w, norm_groups, eps, state, heads,
+                    groups, dim, vdim, out):
+        """Per request, token by token: the convolution over the kept last inputs and the new one (plus its
+        bias), SiLU, rounded to out's dtype; dt = softplus(d + dt_bias); S <- exp(-rate dt) S + x (dt B)^T (S
+        [vdim, dim]); y = S C + skip x; then y * silu(z), divided by the root mean square of its part, times norm_w."""
+        b = ctx.batch
+        cz, cx, cd = cols
+        H, G, N, P = heads, groups, dim, vdim
+        inner, taps = H * P, conv_w.shape[1]
+        C = inner + 2 * G * N
+        n_state = inner * N
+        cu, slots = b.cu_q.tolist(), b.slots.tolist()
+        for r, slot in enumerate(slots):
+            if slot < 0:
+                out[cu[r]:cu[r + 1]] = 0
+                continue
+            S = state[slot, :n_state].reshape(H, P, N).clone()
+            kept = state[slot, n_state:].reshape(taps - 1, C).clone()
+            for t in range(cu[r], cu[r + 1]):
+                window = torch.cat([kept, proj[t, cx:cx + C][None, :]], 0)          # [taps, C], oldest first
+                kept = window[1:]
+                a = (window * conv_w.t()).sum(0) + (conv_b if conv_b is not None else 0.0)
+                a = (a / (1.0 + torch.exp(-a))).to(out.dtype).float()
+                x = a[:inner].reshape(H, P)
+                B = a[inner:inner + G * N].reshape(G, N).repeat_interleave(H // G, 0)
+                Cv = a[inner + G * N:].reshape(G, N).repeat_interleave(H // G, 0)
+                dt = torch.nn.functional.softplus(proj[t, cd:cd + H] + dt_bias)
+                S = torch.exp(-rate * dt)[:, None, None] * S + (dt[:, None] * x)[:, :, None] * B[:, None, :]
+                y = (torch.einsum("hpn,hn->hp", S, Cv) + skip[:, None] * x).reshape(-1)
+                z = proj[t, cz:cz + inner]
+                y = (y * z * torch.sigmoid(z)).reshape(norm_groups, -1)
+                y = y / torch.sqrt((y * y).mean(-1, keepdim=True) + eps)
+                out[t] = (y.reshape(-1) * norm_w).to(out.dtype)
+            state[slot, :n_state] = S.reshape(-1)
+            state[slot, n_state:] = kept.reshape(-1)
+
     # ---- the generalized delta rule ----
     def general_delta(self, ctx, proj, cols, zdec, w0, a0, decay_scale, norm_w, eps, state, heads, dim, vdim, out):
         """Per request, token by token: w = exp(-c sigmoid(zdec + w0)), a = sigmoid(logit + a0), u the
@@ -438,9 +492,10 @@ class CpuOps:
 
     # ---- normed queries and keys; sublayers whose outputs are normed ----
     def qk_norm_rope_append(self, src, cols, q_out, k_pool, v_pool, positions, token_req, block_table, heads, kv_heads,
-                            dim, vdim, q_weight, k_weight, eps, rotary, page_size):
-        """queries and keys normed per head (weights 32-bit; None: not), rotated, queries out, keys and
-        the untouched value columns into their pages"""
+                            dim, vdim, q_weight, k_weight, eps, rotary, page_size, query_growth=None):
+        """queries and keys normed per head (weights 32-bit; None: not), rotated, queries (times 1 + coef
+        ln(floor((p + 1) / every) + 1) at position p with query_growth = (coef, every)) out, keys and
+        the untouched value columns into their pages; kv_heads 0: queries only"""
         T = src.shape[0]
         cq, ck, cv = cols
         q = src[:, cq:cq + heads * dim].float().reshape(T, heads, dim)
@@ -452,7 +507,13 @@ class CpuOps:
             k = k / torch.sqrt((k * k).mean(-1, keepdim=True) + eps) * k_weight
         if rotary is not None:
             q, k = self._rotate(q, positions, rotary), self._rotate(k, positions, rotary)
+        if query_growth is not None:
+            coef, every = query_growth
+            steps = torch.floor((positions.double() + 1.0) / every)
+            q = q * (1.0 + coef * torch.log(steps + 1.0)).float()[:, None, None]
         q_out.copy_(q.to(q_out.dtype))
+        if kv_heads == 0:
+            return
         for t in range(T):
             pos = int(positions[t])
             page = int(block_table[int(token_req[t]), pos // page_size])
@@ -470,6 +531,8 @@ class CpuOps:
             return torch.relu(z) ** 2
         if kind == "tanh":
             return torch.tanh(z)
+        if kind == "gelu":
+            return 0.5 * z * (1.0 + torch.erf(z * 0.5 ** 0.5))
         raise ValueError(kind)
 
     def gate_mul(self, x, gate, kind="sigmoid"):
