@@ -1,0 +1,557 @@
+"""Fosovik on the GPU: every new kernel against its plain reference at sizes of its own, then
+bin/trace_run replaying requests whole, decoded token by token, in portions and mixed with pages and
+slots used again, in 32-bit and bfloat16, against the plain model; a key far back that two layers put their
+weight on; greedy generation through ``Engine.generate`` (graphs, steps launched ahead) and the command
+line; configurations drawn at random."""
+import numpy as np
+import pytest
+import torch
+
+from tests import helpers
+from tests.helpers import TraceRunner
+from tests.fosovik_cases import CASES, SHARPEN, model_dir, plain_logits, random_tokens, weights
+
+pytestmark = pytest.mark.gpu
+
+STORE = {"float32": torch.float32, "bfloat16": torch.bfloat16}
+
+
+def up64(n):
+    return (n + 63) // 64 * 64
+
+
+class _Batch:
+    pass
+
+
+class _Ctx:
+    def __init__(self, device="cuda:0"):
+        from garuda_b200.engine.batch import Workspace
+        self.ws = Workspace(torch.device(device))
+        self.batch = _Batch()
+
+
+@pytest.fixture(scope="module", params=["float32", "bfloat16"])
+def both(request):
+    from garuda_b200.kernels.ops import CudaOps
+    from tests.plain.cpu_ops import CpuOps
+    dt = STORE[request.param]
+    return CudaOps("cuda:0", tensor_cores=dt == torch.bfloat16), CpuOps(), dt
+
+
+def rnd(*shape, dtype=torch.float32, scale=1.0, seed=0):
+    g = torch.Generator().manual_seed(hash((shape, seed)) % (1 << 31))
+    return (torch.randn(*shape, generator=g) * scale).to(dtype)
+
+
+def close(got, want, dt, what, tol=None):
+    got, want = got.float().cpu(), want.float()
+    tol = tol or (2e-2 if dt == torch.bfloat16 else 2e-5)
+    err = (got - want).abs().max().item() / max(want.abs().max().item(), 1e-6)
+    assert torch.isfinite(got).all() and err <= tol, f"{what}: {err:.2e}"
+
+
+def step_batch(lens, starts, slots, page_size, seed=1):
+    """A batch of requests that bring ``lens`` tokens from positions ``starts``, their pages drawn at
+    random from the pool; returns (batch, block table, pages in the pool)."""
+    b = _Batch()
+    R = len(lens)
+    b.cu_q = torch.tensor([0] + list(np.cumsum(lens)), dtype=torch.int32)
+    b.kv_lens = torch.tensor([s + n for s, n in zip(starts, lens)], dtype=torch.int32)
+    b.positions = torch.tensor(np.concatenate([np.arange(s, s + n) for s, n in zip(starts, lens)]), dtype=torch.int32)
+    b.slots = torch.tensor(slots, dtype=torch.int32)
+    b.token_req = torch.repeat_interleave(torch.arange(R, dtype=torch.int32), torch.tensor(lens))
+    b.num_requests, b.max_q_len, b.min_q_len = R, max(lens), min(lens)
+    b.num_tokens, b.max_kv_len = sum(lens), int(b.kv_lens.max())
+    width = (b.max_kv_len + page_size - 1) // page_size + 1
+    table = -torch.ones(R, width, dtype=torch.int32)
+    perm = np.random.default_rng(seed).permutation(R * width)
+    at = 0
+    for r in range(R):
+        n = (int(b.kv_lens[r]) + page_size - 1) // page_size
+        table[r, :n] = torch.tensor(perm[at:at + n], dtype=torch.int32)
+        at += n
+    return b, table, R * width
+
+
+def batches(b):
+    ctx_g, ctx_r = _Ctx(), _Ctx("cpu")
+    ctx_r.batch = b
+    bg = _Batch()
+    for k, v in vars(b).items():
+        setattr(bg, k, v.cuda() if torch.is_tensor(v) else v)
+    ctx_g.batch = bg
+    return ctx_g, ctx_r
+
+
+# ---------------------------------------------------------------------------- kernels
+@pytest.mark.parametrize("T,d", [(1, 44), (37, 200), (5, 1030), (3, 4096), (700, 15)])
+def test_norm_without_statistics(both, T, d):
+    ops, ref, dt = both
+    x, w, b = rnd(T, d, scale=3.0, seed=1), rnd(d, seed=2), rnd(d, seed=3)
+    for rows in (None, torch.tensor([T - 1, 0, T // 2], dtype=torch.int32)):
+        n = T if rows is None else 3
+        want, got = torch.empty(n, d, dtype=dt), torch.empty(n, d, dtype=dt, device="cuda")
+        ref.dynamic_tanh(x, 0.7, w, b, want, rows)
+        ops.dynamic_tanh(x.cuda(), 0.7, w.cuda(), b.cuda(), got, None if rows is None else rows.cuda())
+        close(got, want, dt, f"dynamic_tanh {T}x{d}", 1e-2 if dt == torch.bfloat16 else 3e-6)
+
+
+@pytest.mark.parametrize("H,G,dim,vdim", [(4, 2, 24, 40), (3, 1, 15, 9), (8, 8, 64, 32), (2, 2, 300, 16)])
+@pytest.mark.parametrize("growth", [None, (0.5, 7), (-0.3, 64), (2.0, 1)])
+def test_queries_that_grow_and_normed_keys_into_pages(both, H, G, dim, vdim, growth):
+    """Positions on both sides of every step of the growth; queries alone for a layer that reads
+    another's keys."""
+    ops, ref, dt = both
+    ps = 8
+    b, table, pages = step_batch([5, 1, 60, 2], [0, 62, 3, 5], [2, 0, 3, 1], ps)
+    bg = batches(b)[0].batch
+    T, cols = b.num_tokens, H * dim + G * (dim + vdim)
+    row = rnd(T, cols + 3, seed=1)
+    ones = torch.ones(H, dim)
+    for kv in (G, 0):
+        kp, vp = torch.zeros(pages, G, ps, dim, dtype=dt), torch.zeros(pages, G, ps, vdim, dtype=dt)
+        q = torch.zeros(T, H, dim, dtype=dt)
+        kg, vg, qg = kp.cuda(), vp.cuda(), q.cuda()
+        c = (1, 1 + H * dim, 1 + (H + G) * dim)
+        ref.qk_norm_rope_append(row, c, q, kp, vp, b.positions, b.token_req, table, H, kv, dim, vdim, ones, ones[0], 1e-5, None, ps, query_growth=growth)
+        ops.qk_norm_rope_append(row.cuda(), c, qg, kg, vg, bg.positions, bg.token_req, table.cuda(), H, kv, dim, vdim, ones.cuda(),
+                                ones[0].cuda(), 1e-5, None, ps, query_growth=growth)
+        for got, want, what in ((qg, q, "queries"), (kg, kp, "keys"), (vg, vp, "values")):
+            if kv == 0 and what != "queries":
+                assert not got.any()
+            else:
+                close(got, want, dt, f"{what}, growth {growth}", 1e-2 if dt == torch.bfloat16 else 3e-6)
+
+
+@pytest.mark.parametrize("T,E,K,F,top,N", [(1, 5, 44, 24, 2, 44), (9, 4, 128, 64, 4, 128), (150, 12, 192, 72, 3, 200), (700, 8, 256, 128, 3, 136),
+                                          (65, 3, 64, 200, 1, 72)])
+@pytest.mark.parametrize("kind", ["gelu", "relu2", "silu"])
+def test_experts_without_a_gate(both, T, E, K, F, top, N, kind):
+    """Few pairs, many pairs and the plain kernel; experts nobody chose; the sum added to what is there."""
+    ops, ref, dt = both
+    h, up, down = rnd(T, K, dtype=dt, seed=1), rnd(E, F, K, dtype=dt, scale=0.3, seed=2), rnd(E, N, F, dtype=dt, scale=0.3, seed=3)
+    g = torch.Generator().manual_seed(4)
+    ids = torch.stack([torch.randperm(max(E - 1, top), generator=g)[:top] for _ in range(T)]).to(torch.int32)
+    wts, x = torch.rand(T, top, generator=g), rnd(T, N, seed=5)
+    for scale_input in (False, True):
+        ctx_g, ctx_r = _Ctx(), _Ctx("cpu")
+        want, got = x.clone(), x.clone().cuda()
+        ref.routed_feed_forward(ctx_r, h, up, down, ids, wts, want, kind, 0.0, 0.5, scale_input=scale_input, gated=False)
+        ops.routed_feed_forward(ctx_g, h.cuda(), up.cuda(), down.cuda(), ids.cuda(), wts.cuda(), got, kind, 0.0, 0.5, scale_input=scale_input,
+                                gated=False)
+        close(got, want, dt, f"experts {kind}")
+
+
+@pytest.mark.parametrize("M,N,K", [(21, 77, 40), (3, 320, 160), (300, 1024, 256), (2048, 512, 128)])
+def test_exact_gelu_behind_a_product(both, M, N, K):
+    ops, ref, dt = both
+    a, w = rnd(M, K, dtype=dt, seed=1), rnd(N, K, dtype=dt, scale=0.3, seed=2)
+    ctx_g, ctx_r = _Ctx(), _Ctx("cpu")
+    want, got = torch.empty(M, N, dtype=dt), torch.empty(M, N, dtype=dt, device="cuda")
+    ref.linear_act(ctx_r, a, w, want, "gelu")
+    ops.linear_act(ctx_g, a.cuda(), w.cuda(), got, "gelu")
+    close(got, want, dt, "linear_act gelu")
+
+
+def _ssm(H, G, N, P, taps, parts, T, slots, seed=1, bias=True):
+    """Weights, rows and states of a state space: decays from nearly one to nearly zero."""
+    inner = H * P
+    C = inner + 2 * G * N
+    w = dict(conv_w=rnd(C, taps, scale=0.6, seed=seed), conv_b=rnd(C, scale=0.3, seed=seed + 1) if bias else None,
+             rate=torch.exp(torch.linspace(-4.0, 2.5, H)), dt_bias=rnd(H, scale=0.7, seed=seed + 2), skip=rnd(H, seed=seed + 3),
+             norm_w=rnd(inner, seed=seed + 4))
+    proj = rnd(T, 2 * inner + 2 * G * N + H + 5, seed=seed + 5)
+    cols = (1, inner + 1, inner + C + 2)
+    state = rnd(slots, inner * N + (taps - 1) * C, seed=seed + 6)
+    return w, proj, cols, state, inner, C
+
+
+def _run_ssm(ops, ctx, w, proj, cols, parts, state, H, G, N, P, out, dev):
+    to = (lambda v: None if v is None else v.to(dev))
+    ops.state_space(ctx, proj.to(dev), cols, to(w["conv_w"]), to(w["conv_b"]), to(w["rate"]), to(w["dt_bias"]), to(w["skip"]), to(w["norm_w"]),
+                    parts, 1e-5, state, H, G, N, P, out)
+
+
+SSM_SIZES = [(6, 3, 10, 9, 3, 6), (4, 2, 64, 32, 4, 1), (2, 1, 128, 64, 2, 2), (3, 3, 16, 48, 1, 3), (2, 2, 256, 16, 5, 1), (1, 1, 80, 16, 4, 1),
+             (4, 1, 48, 32, 16, 4), (2, 1, 260, 8, 4, 2), (5, 5, 33, 20, 7, 1)]
+
+
+@pytest.mark.parametrize("H,G,N,P,taps,parts", SSM_SIZES)
+@pytest.mark.parametrize("lens,slots", [([5, 1, 200, 64, 65], [2, 0, 5, 3, 1]), ([1, 1, 1], [1, 4, 0]), ([2, 3], [0, 1]), ([129], [3]), ([17, 23, 1], [3, 0, 1])])
+def test_state_space_steps(both, H, G, N, P, taps, parts, lens, slots):
+    """Mixed steps (single tokens beside portions that end inside a chunk, at its edge and just behind), single
+    tokens alone, short portions; states that are not zero; a slot nobody uses is left as it is, NaN and all."""
+    ops, ref, dt = both
+    b, _, _ = step_batch(lens, [3] * len(lens), slots, 8)
+    ctx_g, ctx_r = batches(b)
+    T = b.num_tokens
+    w, proj, cols, state, inner, C = _ssm(H, G, N, P, taps, parts, T, 7)
+    state[6] = float("nan")
+    want, s_want = torch.zeros(T, inner, dtype=dt), state.clone()
+    _run_ssm(ref, ctx_r, w, proj, cols, parts, s_want, H, G, N, P, want, "cpu")
+    got, s_got = torch.zeros(T, inner, dtype=dt, device="cuda"), state.clone().cuda()
+    _run_ssm(ops, ctx_g, w, proj, cols, parts, s_got, H, G, N, P, got, "cuda")
+    close(got, want, dt, f"state space {lens}", 2e-2 if dt == torch.bfloat16 else 5e-5)
+    assert torch.isnan(s_got[6]).all()
+    # the state takes the rounded activations in both: what differs is 32-bit rounding (and a rounding to bfloat16
+    # that falls the other way here and there)
+    close(s_got[:6], s_want[:6], torch.float32, "its state", 4e-3 if dt == torch.bfloat16 else 5e-5)
+
+
+def test_state_space_padding_rows_touch_no_state(both):
+    ops, ref, dt = both
+    H, G, N, P, taps, parts = 4, 2, 64, 32, 4, 1
+    b, _, _ = step_batch([1, 1, 1, 1], [3, 3, 0, 0], [1, 0, -1, -1], 8)
+    ctx_g, ctx_r = batches(b)
+    w, proj, cols, state, inner, C = _ssm(H, G, N, P, taps, parts, 4, 3)
+    want, s_want = torch.zeros(4, inner, dtype=dt), state.clone()
+    _run_ssm(ref, ctx_r, w, proj, cols, parts, s_want, H, G, N, P, want, "cpu")
+    got, s_got = torch.zeros(4, inner, dtype=dt, device="cuda"), state.clone().cuda()
+    _run_ssm(ops, ctx_g, w, proj, cols, parts, s_got, H, G, N, P, got, "cuda")
+    close(got[:2], want[:2], dt, "rows with a slot", 2e-2 if dt == torch.bfloat16 else 5e-5)
+    assert torch.equal(s_got[2].cpu(), state[2])
+
+
+@pytest.mark.parametrize("H,G,N,P", [(4, 2, 64, 32), (2, 1, 128, 64), (2, 1, 256, 16)])
+def test_chunks_on_the_tensor_cores_keep_32_bit_states(H, G, N, P):
+    """700 tokens through the chunked kernel, through the token-by-token kernel and in steps of many sizes: the same
+    rounded activations enter all three, so states and outputs agree to 32-bit rounding, far below
+    bfloat16's (a state or a weight rounded to bfloat16 anywhere would differ by 2^-9)."""
+    from garuda_b200.kernels.ops import CudaOps
+    ops = CudaOps("cuda:0")
+    taps, parts, T = 4, 1, 700
+    w, proj, cols, state, inner, C = _ssm(H, G, N, P, taps, parts, T, 2)
+    w["rate"] = torch.exp(torch.linspace(-6.0, 1.0, H))            # long memories among them
+    ys, states = [], []
+    for cut in ([T], [T], (1, 2, 23, 24, 64, 65, 1, 300, 1, 219)):
+        st, outs, at = state.clone().cuda(), [], 0
+        ops.SSD_CHUNK_TOKENS = 10 ** 9 if len(ys) == 1 else 24
+        for n in cut:
+            b, _, _ = step_batch([n], [at], [1], 8)
+            ctx, _ = batches(b)
+            out = torch.zeros(n, inner, dtype=torch.bfloat16, device="cuda")
+            _run_ssm(ops, ctx, w, proj[at:at + n], cols, parts, st, H, G, N, P, out, "cuda")
+            outs.append(ctx.ws.get("ssd_y", (n, inner), torch.float32).clone())        # before the norm and its rounding
+            at += n
+        assert at == T
+        ys.append(torch.cat(outs))
+        states.append(st)
+    for k in (1, 2):
+        close(ys[k], ys[0].cpu(), torch.float32, "outputs", 2e-5)
+        close(states[k][1], states[0][1].cpu(), torch.float32, "states", 2e-5)
+    assert torch.equal(states[0][0].cpu(), state[0])
+
+
+# ---------------------------------------------------------------------------- the engine, replayed
+def check(got, ref, dtype, what, name):
+    """Per position, the largest difference as a fraction of the largest logit. 32-bit: every position
+    within 2e-4 (sums in another order than the 64-bit plain model's). bfloat16: nine positions in ten
+    within 0.05 and the median within 0.015, the rest finite: with sharpened random weights a router's
+    close call or a sharp softmax turns the rounding of an input into a large change at a few positions,
+    in the plain model itself; a fault of a kernel, a mask or a state shows at most positions."""
+    scale = float(np.abs(ref).max())
+    assert got.shape == ref.shape and np.isfinite(got).all(), what
+    err = np.abs(got - ref).max(-1) / scale
+    helpers.OBSERVED[f"{name}/{dtype}"] = max(helpers.OBSERVED.get(f"{name}/{dtype}", 0.0), float(np.median(err)))
+    if dtype == "float32":
+        assert err.max() <= 2e-4, f"{what}: {err.max():.3e} of the largest logit at position {int(err.argmax())}"
+        return
+    over = int((err > 0.05).sum())
+    assert over <= max(1, len(err) // 10), f"{what}: {over} of {len(err)} positions beyond 0.05 (largest {err.max():.3e})"
+    assert np.median(err) <= 0.015, f"{what}: median {np.median(err):.3e}"
+
+
+@pytest.fixture(scope="module", params=[(n, d) for n in CASES for d in ("float32", "bfloat16")], ids=lambda p: f"{p[0]}-{p[1]}")
+def run(request):
+    name, dtype = request.param
+    tr = TraceRunner(model_dir(name, STORE[dtype]), dtype, max_tokens=4 * up64(130), extra=["--page-size", "16"])
+    yield name, dtype, tr
+    assert tr.close() == 0
+
+
+def test_whole(run):
+    name, dtype, tr = run
+    for n, seed in ((1, 1), (2, 2), (17, 3), (130, 4)):
+        toks = random_tokens(name, n, seed)
+        out = tr.step([("w", toks, range(n))], end=["w"])
+        check(out, plain_logits(name, STORE[dtype], toks), dtype, f"whole, {n} tokens", name)
+
+
+def test_prompt_then_token_by_token(run):
+    name, dtype, tr = run
+    toks = random_tokens(name, 120, 7)
+    ref = plain_logits(name, STORE[dtype], toks)
+    outs = [tr.step([("d", toks[:39], [38])])]
+    for i in range(39, 120):                      # every step of the queries' growth is passed by decoded tokens
+        outs.append(tr.step([("d", [toks[i]], [0])], end=["d"] if i == 119 else []))
+    check(np.concatenate(outs), ref[38:], dtype, "decode after a prompt", name)
+
+
+def test_long_decoding_from_the_first_token(run):
+    name, dtype, tr = run
+    toks = random_tokens(name, 100, 9)
+    ref = plain_logits(name, STORE[dtype], toks)
+    got = np.concatenate([tr.step([("l", [t], [0])], end=["l"] if i == 99 else []) for i, t in enumerate(toks)])
+    check(got[:4], ref[:4], dtype, "first tokens", name)
+    check(got, ref, dtype, "long decoding", name)
+
+
+def test_portions_down_to_two_tokens(run):
+    name, dtype, tr = run
+    toks = random_tokens(name, 118, 11)
+    ref = plain_logits(name, STORE[dtype], toks)
+    cuts = [7, 2, 19, 3, 2, 16, 2, 31, 1, 15, 2, 18]
+    pos, outs = 0, []
+    for i, c in enumerate(cuts):
+        outs.append(tr.step([("p", toks[pos:pos + c], range(c))], end=["p"] if i == len(cuts) - 1 else []))
+        pos += c
+    assert pos == 118
+    check(np.concatenate(outs), ref, dtype, "portions", name)
+
+
+def test_mixed_requests_reusing_pages_and_slots(run):
+    name, dtype, tr = run
+    lens = [90, 33, 128, 21, 64, 2, 75]
+    toks = [random_tokens(name, n, 20 + i) for i, n in enumerate(lens)]
+    refs = [plain_logits(name, STORE[dtype], t) for t in toks]
+    pool = 4 * up64(130) - 128
+    fed, got = [0] * len(lens), [[] for _ in lens]
+    live, waiting = [], list(range(len(lens)))
+    rng = np.random.default_rng(1)
+    most = 0
+    while live or waiting:
+        while waiting and len(live) < 4 and sum(up64(lens[i]) for i in live) + up64(lens[waiting[0]]) <= pool:
+            live.append(waiting.pop(0))
+        most = max(most, len(live))
+        entries, ended = [], []
+        active = [i for i in live if rng.random() > 0.15] or live[:1]        # now and then a request sits a step out
+        for i in active:
+            left = lens[i] - fed[i]
+            n = 1 if left <= 12 else int(min(left - 12, rng.integers(2, 24)))
+            entries.append((f"m{i}", toks[i][fed[i]:fed[i] + n], range(n)))
+            if fed[i] + n == lens[i]:
+                ended.append(f"m{i}")
+        out = tr.step(entries, end=ended)
+        row = 0
+        for (_, t, _), i in zip(entries, active):
+            got[i].append(out[row:row + len(t)])
+            row += len(t)
+            fed[i] += len(t)
+            if fed[i] == lens[i]:
+                live.remove(i)
+    assert most == 4
+    for i in range(len(lens)):
+        check(np.concatenate(got[i]), refs[i], dtype, f"mixed, request {i}", name)
+
+
+def test_every_way_of_cutting_gives_the_same_logits_in_32_bit(run):
+    name, dtype, tr = run
+    if dtype != "float32":
+        pytest.skip("compared against the plain model in bfloat16")
+    toks = random_tokens(name, 80, 31)
+    whole = tr.step([("x", toks, range(80))], end=["x"])
+    parts = [tr.step([("y", toks[:50], range(50))])]
+    parts += [tr.step([("y", [t], [0])]) for t in toks[50:79]]
+    parts.append(tr.step([("y", [toks[79]], [0])], end=["y"]))
+    assert np.abs(np.concatenate(parts) - whole).max() <= 2e-5 * max(1.0, np.abs(whole).max())
+
+
+def _planted(tmp_path, dtype):
+    """A model in which a query of token 1 finds the key of token 0, wherever it is, in a layer of its own and in
+    another that reads the first one's keys: unit queries and keys on one shared channel, a scale of 9."""
+    from garuda_b200.weights import SafetensorsFolder, write_random_model, write_safetensors
+    from tests.fosovik_cases import _att, _dense, _layer, _ssm as ssm_cfg
+    import json
+    cfg = {"architecture": "Fosovik", "vocab": 80, "width": 48, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+           "layers": [_layer("attention", _att(2, 1, 16, 32, 9.0, temp=(0.2, 50)), None),
+                      _layer("mamba2", ssm_cfg(2, 16, 16, 1, 4, 1), _dense(32, 1.0)),
+                      _layer("attention", _att(2, 1, 16, 32, 9.0, kv_from=0), None)]}
+    d = write_random_model(str(tmp_path / dtype), cfg, 3, store_dtype=STORE[dtype], scale={"mix.v": 8.0, "mix.o": 12.0, "embed": 10.0, "head": 8.0})
+    f = SafetensorsFolder(d)
+    t = {n: f.tensor(n).clone() for n in f.names()}
+    t["embed"][:, :2] = 0.0
+    t["embed"][0], t["embed"][1] = 0.0, 0.0
+    t["embed"][0, 0], t["embed"][1, 1] = 6.0, 6.0
+    for n in ("l0", "l2"):
+        t[n + ".norm1.b"][:2] = 0.0
+        t[n + ".norm1.b"] *= 0.1
+        q = t[n + ".mix.q"].view(2, 16, 48)
+        q[:, :, :2] = 0.0
+        q[:, 0, :] = 0.0
+        q[:, 0, 1] = 40.0
+    k = t["l0.mix.k"]
+    k[:, :2] = 0.0
+    k[0, :] = 0.0
+    k[0, 0] = 40.0
+    write_safetensors(d + "/model.safetensors", t)
+    return d, cfg
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_a_key_far_back_that_two_layers_read(dtype, tmp_path):
+    """Token 0 once, at places on page borders and beside them, hundreds of positions in front of the queries (token 1),
+    which stand in a portion and are decoded; without the far key the plain model's logits are others altogether."""
+    from tests.plain import fosovik_plain as fp
+    d, cfg = _planted(tmp_path, dtype)
+    W = helpers.folder_weights(d)
+    tr = TraceRunner(d, dtype, max_tokens=up64(640), extra=["--page-size", "16"])
+    base = np.random.default_rng(5).integers(2, 80, 601)
+    for k, at in enumerate((0, 1, 15, 16, 31, 255)):
+        toks = base.copy()
+        toks[at] = 0
+        toks[[598, 600]] = 1
+        ref = fp.forward(cfg, W, toks).astype(np.float32)
+        toks2 = toks.copy()
+        toks2[at] = base[at]
+        other = fp.forward(cfg, W, toks2).astype(np.float32)
+        scale = np.abs(ref).max()
+        assert np.abs(other[600] - ref[600]).max() > 0.2 * scale, "the far key does not show"
+        toks = toks.tolist()
+        tr.step([(f"a{k}", toks[:300], [])])
+        out = [tr.step([(f"a{k}", toks[300:599], [298])])]
+        out += [tr.step([(f"a{k}", [t], [0])], end=[f"a{k}"] if i == 1 else []) for i, t in enumerate(toks[599:])]
+        err = np.abs(np.concatenate(out) - ref[598:]).max(-1) / scale
+        assert err.max() <= (1e-4 if dtype == "float32" else 0.04), f"far key at {at}: {err}"
+    assert tr.close() == 0
+
+
+def test_a_long_request_whose_early_tokens_reach_the_end():
+    """700 tokens; the last logits follow the plain model in both dtypes, and they change with token 3."""
+    name = "FD"
+    toks = random_tokens(name, 700, 3)
+    for dtype in ("float32", "bfloat16"):
+        ref = plain_logits(name, STORE[dtype], toks)
+        tr = TraceRunner(model_dir(name, STORE[dtype]), dtype, max_tokens=up64(700))
+        tr.step([("a", toks[:300], [])])
+        out = tr.step([("a", toks[300:], range(390, 400))], end=["a"])
+        check(out, ref[690:], dtype, "the end of 700 tokens", name)
+        if dtype == "float32":
+            other = list(toks)
+            other[3] = (toks[3] + 1) % CASES[name][0]["vocab"]
+            alt = tr.step([("b", other, range(690, 700))], end=["b"])
+            assert np.abs(alt - out).max() > 1e-4 * np.abs(out).max()
+        assert tr.close() == 0
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_greedy_generation_through_the_engine(dtype):
+    from garuda_b200 import Engine, SamplingParams
+    from tests.plain import fosovik_plain as fp
+    name = "FB"
+    cfg, w = CASES[name][0], weights(name, STORE[dtype])
+    e = Engine(model_dir(name, STORE[dtype]), dtype=dtype, context=256, kv_tokens=1024, max_concurrent=4)
+    assert e.model.graph_safe
+    prompts = [random_tokens(name, n, 70 + n) for n in (5, 40, 1, 23, 64)]
+    res = e.generate(prompts, SamplingParams.greedy(max_tokens=12))
+    assert e.runner.graphs.replays > 0
+    for p, r in zip(prompts, res):
+        assert r.finish_reason == "length" and len(r.tokens) == 12
+        seq = list(p)
+        for tok in r.tokens:
+            logits = fp.forward(cfg, w, seq)[-1]
+            slack = (1e-4 if dtype == "float32" else 0.05) * float(np.abs(logits).max())
+            assert logits[tok] >= float(logits.max()) - slack, f"token {tok} has logit {logits[tok]}, the best is {logits.max()}"
+            seq.append(tok)
+
+
+# ---------------------------------------------------------------------------- configurations drawn at random
+def _random_config(rng):
+    def pick(xs):
+        return xs[int(rng.integers(0, len(xs)))]
+
+    g, dim, vdim = pick([1, 2, 3]), pick([8, 12, 15, 32, 64, 128]), pick([8, 20, 32, 64, 128])     # layers that share keys agree on these
+
+    def attention(sources):
+        m = {"heads": g * pick([1, 2, 4]), "kv_heads": g, "dim": dim, "vdim": vdim, "scale": pick([0.3, 0.6, 1.0])}
+        if pick([True, True, False]):
+            m["q_temp"] = {"coef": pick([0.1, 0.5, -0.1]), "every": pick([1, 5, 16, 64])}
+        if sources and pick([True, False]):
+            m["kv_from"] = pick(sources)
+        return {"type": "attention", "mixer": m}
+
+    def recurrence():
+        groups = pick([1, 2, 3])
+        heads, width = groups * pick([1, 2, 3]), pick([8, 16, 20, 32, 64])
+        parts = pick([1, groups, heads])
+        return {"type": "mamba2", "mixer": {"heads": heads, "vdim": width, "state": pick([4, 16, 33, 64, 128, 144]), "groups": groups,
+                                            "conv": pick([1, 2, 3, 4, 7]), "norm_groups": parts}}
+
+    def mlp():
+        kind = pick(["dense", "dense", "moe", "moe", None])
+        if kind == "dense":
+            return {"kind": "dense", "ff": pick([8, 24, 56, 128]), "limit": pick([0.5, 1.5, 7.0])}
+        if kind == "moe":
+            experts = pick([1, 2, 5, 12, 33])
+            return {"kind": "moe", "expert": {"ff": pick([8, 24, 64])}, "router": {"experts": experts, "top": int(rng.integers(1, min(experts, 6) + 1))}}
+        return None
+
+    layers, sources = [], []
+    for i in range(pick([1, 2, 3, 5])):
+        layer = dict(attention(sources) if pick([True, False]) else recurrence(), mlp=mlp())
+        if layer["type"] == "attention" and "kv_from" not in layer["mixer"]:
+            sources.append(i)
+        layers.append(layer)
+    return {"architecture": "Fosovik", "vocab": pick([50, 97, 300, 1000]), "width": pick([40, 64, 72, 136, 256]),
+            "embedding": {"scale": pick([1.0, 3.0, 12.0])}, "norm": {"eps": pick([1e-5, 1e-6])}, "layers": layers}
+
+
+@pytest.mark.parametrize("seed", [2, 5, 11, 17])
+def test_configurations_drawn_at_random(seed, tmp_path):
+    from garuda_b200.weights import write_random_model
+    from tests.plain import fosovik_plain as fp
+    rng = np.random.default_rng(seed)
+    for k in range(3):
+        cfg = _random_config(rng)
+        for dtype in ("float32", "bfloat16"):
+            d = write_random_model(str(tmp_path / f"m{k}{dtype}"), cfg, seed * 10 + k, store_dtype=STORE[dtype], scale=SHARPEN)
+            w = helpers.folder_weights(d)
+            a, b = rng.integers(0, cfg["vocab"], 70).tolist(), rng.integers(0, cfg["vocab"], 45).tolist()
+            ra, rb = fp.forward(cfg, w, a).astype(np.float32), fp.forward(cfg, w, b).astype(np.float32)
+            tr = TraceRunner(d, dtype, max_tokens=2 * up64(70), extra=["--page-size", "16"])
+            check(tr.step([("w", a, range(70))], end=["w"]), ra, dtype, f"seed {seed}.{k}: whole", "random")
+            outs_a, outs_b = [tr.step([("a", a[:40], range(40)), ("b", b[:3], range(3))])], []
+            outs_b.append(outs_a[0][40:])
+            outs_a[0] = outs_a[0][:40]
+            o = tr.step([("b", b[3:30], range(27)), ("a", a[40:42], range(2))])
+            outs_b.append(o[:27])
+            outs_a.append(o[27:])
+            for i in range(15):
+                o = tr.step([("a", [a[42 + i]], [0]), ("b", [b[30 + i]], [0])], end=["b"] if i == 14 else [])
+                outs_a.append(o[:1])
+                outs_b.append(o[1:])
+            outs_a.append(tr.step([("a", a[57:], range(13))], end=["a"]))
+            check(np.concatenate(outs_a), ra, dtype, f"seed {seed}.{k}: request a", "random")
+            check(np.concatenate(outs_b), rb, dtype, f"seed {seed}.{k}: request b", "random")
+            assert tr.close() == 0
+
+
+def test_command_line_generates_with_sampling(tmp_path):
+    """`garuda generate` on a folder of this design: greedy tokens are the plain model's, and a
+    sampled run with a seed (temperature, top-k, top-p through the engine's sampler) repeats itself."""
+    import json
+    import os
+    import subprocess
+    import sys
+    from tests.plain import fosovik_plain as fp
+    name = "FA"
+    d = model_dir(name)
+    cfg = tmp_path / "config.toml"
+    prompt = random_tokens(name, 11, 5)
+    exe = [sys.executable, os.path.join(helpers.ROOT, "bin", "garuda")]
+
+    def generate(sampling, *more):
+        cfg.write_text(f'[model]\npath = "{d}"\ndtype = "float32"\ncontext = 128\n[memory]\npage_size = 16\n[sampling]\n{sampling}')
+        out = subprocess.run(exe + ["--config", str(cfg), "generate", "--prompt-ids", ",".join(map(str, prompt)), *more],
+                             capture_output=True, text=True)
+        assert out.returncode == 0, out.stderr
+        return json.loads(out.stdout.strip().splitlines()[-1])
+
+    rec = generate("temperature = 0.0\nmax_tokens = 6\n")
+    seq = list(prompt)
+    for _ in range(6):
+        seq.append(int(np.argmax(fp.forward(CASES[name][0], weights(name), seq)[-1])))
+    assert rec["tokens"] == seq[len(prompt):] and rec["finish_reason"] == "length"
+    a = generate("temperature = 0.9\ntop_k = 20\ntop_p = 0.9\nmax_tokens = 8\n", "--seed", "4")
+    b = generate("temperature = 0.9\ntop_k = 20\ntop_p = 0.9\nmax_tokens = 8\n", "--seed", "4")
+    assert a["tokens"] == b["tokens"] and len(a["tokens"]) == 8
