@@ -6,7 +6,7 @@
 // s_j = dot(q, K_j) * scale with the scale multiplied after the dot; keys j in
 // [start, pos], start = max(0, pos + 1 - window) (garuda/src/cache/mod.rs:333-338);
 // softmax with the maximum subtracted (garuda/src/simd/mod.rs:132-158); then the
-// sum of p_j V_j in key order. Keys are walked 32 at a time from `start`, with
+// sum of p_j V_j in key order, 32 keys by themselves and the 32s added up. Keys are walked 32 at a time from `start`, with
 // a running maximum and sum, so the result for a token does not depend on what
 // else is in the batch or on how its prompt was cut.
 //
@@ -77,9 +77,14 @@ attention_simple_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, c
     float s = -INFINITY;
     if (row >= 0) {
       const T* kr = k_pool + row * hd;
-      float dot = 0.f;
-      for (int c = 0; c < hd; ++c) dot = fmaf(q_s[warp][c], gb::to_float<T>(kr[c]), dot);
-      s = dot * scale;
+      // eight interleaved sums, added up as a tree: less rounding than one sum of hd terms
+      float d8[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      int c = 0;
+      for (; c + 8 <= hd; c += 8)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) d8[e] = fmaf(q_s[warp][c + e], gb::to_float<T>(kr[c + e]), d8[e]);
+      for (int e = 0; c + e < hd; ++e) d8[0] = fmaf(q_s[warp][c + e], gb::to_float<T>(kr[c + e]), d8[0]);
+      s = (((d8[0] + d8[1]) + (d8[2] + d8[3])) + ((d8[4] + d8[5]) + (d8[6] + d8[7]))) * scale;
       if (softcap > 0.f) s = softcap * tanhf(s / softcap);
       if (r1) s -= far1 * log1pf(far2 * (float)(pos - j));
     }
@@ -89,8 +94,9 @@ attention_simple_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, c
     const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);
     l = l * corr + gb::warp_sum(p);
     m = m_new;
+    float part[MAX_HD / 32];       // the block's keys summed by themselves, then added to the keys in front
 #pragma unroll
-    for (int i = 0; i < MAX_HD / 32; ++i) acc[i] *= corr;
+    for (int i = 0; i < MAX_HD / 32; ++i) part[i] = 0.f;
     const int n_here = min(32, last - base + 1);
     for (int jj = 0; jj < n_here; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
@@ -100,9 +106,11 @@ attention_simple_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, c
 #pragma unroll
       for (int i = 0; i < MAX_HD / 32; ++i) {
         const int c = lane + 32 * i;
-        if (i < nacc && c < vd) acc[i] = fmaf(pj, gb::to_float<T>(vr[c]), acc[i]);
+        if (i < nacc && c < vd) part[i] = fmaf(pj, gb::to_float<T>(vr[c]), part[i]);
       }
     }
+#pragma unroll
+    for (int i = 0; i < MAX_HD / 32; ++i) acc[i] = fmaf(acc[i], corr, part[i]);
   }
   if (sink_v && m != -INFINITY) l += expf(sink_v[h] - m);
   else if (sink && m != -INFINITY) l += expf(-m);

@@ -28,6 +28,15 @@ constexpr int MAX_TAPS = 16;
 __device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
+// A decay a = exp(log_a) as the two numbers that a state is moved on with, S <- keep S + (change S + input). A slow
+// decay (a close to one) is 1 + expm1(log_a): the second term holds what a rounded `a` would lose, which over
+// hundreds of tokens is the larger part of the state's error. A fast one is (a, 0).
+__device__ __forceinline__ void decay_parts(float log_a, float& keep, float& change) {
+  const bool slow = log_a > -0.5f;
+  keep = slow ? 1.0f : expf(log_a);
+  change = slow ? expm1f(log_a) : 0.0f;
+}
+
 // Input of channel c at `lag` tokens before token t (index j within its request's rows of this step): from the
 // step's rows, or from the request's kept inputs [taps - 1, C] (oldest first).
 __device__ __forceinline__ float conv_input(const float* __restrict__ rows, long long P, int t, int j, int lag, int c,
@@ -141,7 +150,8 @@ ssd_recurrence_kernel(const XT* __restrict__ act, int C, const float* __restrict
                       long long state_stride, int H, int G, int dim, int vdim, float* __restrict__ y) {
   gb::pdl_wait();
   constexpr int W = PER * 32;
-  __shared__ float sb[REC_TOKENS][W], sc[REC_TOKENS][W], sx[REC_TOKENS][REC_WARPS * REC_ROWS], sdt[REC_TOKENS], sa[REC_TOKENS];
+  __shared__ float sb[REC_TOKENS][W], sc[REC_TOKENS][W], sx[REC_TOKENS][REC_WARPS * REC_ROWS], sdt[REC_TOKENS];
+  __shared__ float s_keep[REC_TOKENS], s_change[REC_TOKENS];
   const int h = blockIdx.x, r = blockIdx.y, p0 = blockIdx.z * REC_WARPS * REC_ROWS;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int slot = slots[r], t0 = cu_q[r], t1 = cu_q[r + 1];
@@ -173,11 +183,11 @@ ssd_recurrence_kernel(const XT* __restrict__ act, int C, const float* __restrict
     if (threadIdx.x < n) {
       const float* st = step + (size_t)(c0 + threadIdx.x) * 2 * H;
       sdt[threadIdx.x] = st[h];
-      sa[threadIdx.x] = expf(st[H + h]);
+      decay_parts(st[H + h], s_keep[threadIdx.x], s_change[threadIdx.x]);
     }
     __syncthreads();
     for (int tt = 0; tt < n; ++tt) {
-      const float a = sa[tt], dt = sdt[tt];
+      const float keep = s_keep[tt], change = s_change[tt], dt = sdt[tt];
       float acc[REC_ROWS];
 #pragma unroll
       for (int i = 0; i < REC_ROWS; ++i) acc[i] = 0.f;
@@ -186,7 +196,7 @@ ssd_recurrence_kernel(const XT* __restrict__ act, int C, const float* __restrict
         const float b = dt * sb[tt][lane + 32 * k], c = sc[tt][lane + 32 * k];
 #pragma unroll
         for (int i = 0; i < REC_ROWS; ++i) {
-          S[i][k] = fmaf(a, S[i][k], sx[tt][warp * REC_ROWS + i] * b);
+          S[i][k] = fmaf(keep, S[i][k], fmaf(change, S[i][k], sx[tt][warp * REC_ROWS + i] * b));
           acc[i] = fmaf(S[i][k], c, acc[i]);
         }
       }
@@ -263,7 +273,9 @@ ssd_decode_kernel(const Conv cv, const float* __restrict__ d_rows, const float* 
     sm[i] = gb::to_float<XT>(gb::from_float<XT>(v));
   }
   const float dt = softplus(d_rows[(size_t)t * cv.P + h] + dt_bias[h]);
-  const float a = expf(-rate[h] * dt), dskip = skip[h];
+  float keep, change;
+  decay_parts(-rate[h] * dt, keep, change);
+  const float dskip = skip[h];
   __syncthreads();
   float b[QUADS][4], c4[QUADS][4];
 #pragma unroll
@@ -285,7 +297,7 @@ ssd_decode_kernel(const Conv cv, const float* __restrict__ d_rows, const float* 
       for (int q = 0; q < QUADS; ++q) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          S[i][q][e] = fmaf(a, S[i][q][e], x * b[q][e]);
+          S[i][q][e] = fmaf(keep, S[i][q][e], fmaf(change, S[i][q][e], x * b[q][e]));
           acc = fmaf(S[i][q][e], c4[q][e], acc);
         }
         const int c = (lane + q * ROW_LANES) * 4;
