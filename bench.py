@@ -8,6 +8,7 @@
     python bench.py --design murilorn [--size 2k,4k]    (likewise for the third architecture)
     python bench.py --design luvapel [--size 2k,4k]     (the fourth, beside the third)
     python bench.py --design midulorn [--size 2k,4k]    (the fifth, beside the third)
+    python bench.py --design fosovik [--size 2k,4k]     (the sixth, beside the third)
     python bench.py --design kavenex [--size 2k,4k]     (a JSON line of its own: the second architecture
                                                          beside Llama at equal sizes, kernel beside like kernel)
 
@@ -1359,6 +1360,219 @@ def run_design_midulorn(args) -> dict:
     return out
 
 
+# ``--design fosovik``: the Fosovik design beside the Murilorn decoder (the closest of the engine's models: attention
+# with a sink and no position encoding, a recurrence with a matrix of state per head behind short convolutions,
+# routed experts) at equal width, heads, head sizes, state sizes and depth (random weights). Four layers: attention
+# with a dense feed-forward, two state spaces with experts, attention over the first layer's keys with experts.
+FOSOVIK_SIZES = {
+    "2k": dict(width=2048, heads=32, kv_heads=4, dim=64, s_heads=64, s_vdim=64, s_state=128, s_groups=8, s_parts=8, taps=4,
+               ff=5632, experts=16, top=4, expert_ff=1408, vocab=32000, d_heads=32, d_kv_heads=16, d_dim=128, d_vdim=128, rank=64),
+    "4k": dict(width=4096, heads=32, kv_heads=8, dim=128, s_heads=128, s_vdim=64, s_state=128, s_groups=8, s_parts=8, taps=4,
+               ff=11008, experts=16, top=4, expert_ff=2752, vocab=32000, d_heads=64, d_kv_heads=16, d_dim=128, d_vdim=128, rank=128),
+}
+
+
+def fosovik_configs(z):
+    moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["expert_ff"]}}
+    dense = {"kind": "dense", "ff": z["ff"], "limit": 7.0}
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5}
+    grows = dict(att, q_temp={"coef": 0.1, "every": 1024})
+    ssm = {"type": "mamba2", "mlp": moe, "mixer": {"heads": z["s_heads"], "vdim": z["s_vdim"], "state": z["s_state"], "groups": z["s_groups"],
+                                                   "conv": z["taps"], "norm_groups": z["s_parts"]}}
+    fosovik = {"architecture": "Fosovik", "vocab": z["vocab"], "width": z["width"], "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5},
+               "max_positions": 4096, "layers": [{"type": "attention", "mixer": grows, "mlp": dense}, ssm, ssm,
+                                                 {"type": "attention", "mixer": dict(grows, kv_from=0), "mlp": moe}]}
+    attn = {"type": "attention", "mixer": dict(att, softcap=30.0)}
+    delta = {"type": "channel_delta", "mixer": {"heads": z["d_heads"], "kv_heads": z["d_kv_heads"], "dim": z["d_dim"],
+                                                "vdim": z["d_vdim"], "conv": z["taps"], "decay_rank": z["rank"], "gate_rank": z["rank"]}}
+    murilorn = {"architecture": "Murilorn", "vocab": z["vocab"], "width": z["width"], "embedding": {"scale": 1.0},
+                "norm": {"eps": 1e-5}, "streams": 2, "logit_scale": 1.0, "logit_softcap": 30.0, "max_positions": 4096,
+                "layers": [dict(m, mlp=moe) for m in (attn, delta, delta, attn)]}
+    return fosovik, murilorn
+
+
+def run_design_fosovik(args) -> dict:
+    """Prefill and decode throughput of the Fosovik design and of the Murilorn decoder at equal sizes, and
+    the design's kernels beside the like kernels of the engine's other models, each against its roofline (the
+    slower of bytes / measured copy rate and FLOPs / measured bfloat16 rate)."""
+    import numpy as np
+    import torch
+    from types import SimpleNamespace
+    from garuda_b200 import Engine, StepEntry
+    from garuda_b200.engine.batch import Workspace
+    from garuda_b200.weights import write_random_model
+
+    hbm_peak, tflops_peak, peak_kind = peaks()
+    ev = lambda: torch.cuda.Event(enable_timing=True)
+    dev = torch.device("cuda:0")
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+
+    def timed(fn, reps=10):
+        for _ in range(3):
+            fn()
+        times = []
+        for _ in range(reps):
+            flush.zero_()
+            s, e = ev(), ev()
+            torch.cuda.synchronize()
+            s.record()
+            fn()
+            e.record()
+            torch.cuda.synchronize()
+            times.append(s.elapsed_time(e))
+        return sorted(times)[len(times) // 2]
+
+    def roof(ms, flops=0.0, nbytes=0.0):
+        ideal = max(flops / (tflops_peak * 1e12), nbytes / (hbm_peak * 1e9)) * 1e3
+        return {"ms": round(ms, 4), "roofline_ms": round(ideal, 4), "frac": round(ideal / ms, 4)}
+
+    out = {"design": "fosovik", "beside": "murilorn", "peaks": peak_kind, "hbm_gbs": hbm_peak, "bf16_tflops": tflops_peak,
+           "dtype": "bf16", "data": "synthetic",
+           "timing": "CUDA events, 3 warm-up runs, L2 flushed before every timed run, median", "sizes": {}}
+    B, CTX, T = 8, 2048, PREFILL_TOKENS
+    for name in (args.size.split(",") if args.size else list(FOSOVIK_SIZES)):
+        z = FOSOVIK_SIZES[name]
+        rec, engines = {}, {}
+        for arch, cfg in zip(("fosovik", "murilorn"), fosovik_configs(z)):
+            if args.only == "attention" or (args.only and arch == "murilorn"):
+                continue
+            tmp = tempfile.mkdtemp(prefix="garuda_bench_", dir="/dev/shm" if os.path.isdir("/dev/shm") else None)
+            try:
+                write_random_model(tmp, cfg, seed=0, store_dtype=torch.bfloat16)
+                engine = Engine(tmp, dtype="bfloat16", context=4096, page_size=32, kv_tokens=B * CTX + 4096 + 64,
+                                max_concurrent=B, max_batch_tokens=T, prefill_chunk=T, ignore_eos=True)
+            finally:
+                shutil.rmtree(tmp, ignore_errors=True)
+            engines[arch] = engine
+            runner, rng, V = engine.runner, np.random.default_rng(0), z["vocab"]
+            toks = rng.integers(0, V, T).tolist()
+            rid = [0]
+
+            def prefill():
+                rid[0] += 1
+                runner.run([StepEntry(10_000 + rid[0], toks, [T - 1])])
+                runner.end(10_000 + rid[0])
+
+            rec[arch] = {}
+            if args.only != "decode":
+                ms = timed(prefill, reps=5)
+                rec[arch] = {"prefill_2048_ms": round(ms, 3), "prefill_tok_s": round(T / ms * 1e3)}
+            if args.only != "prefill":
+                steps = 48
+                for r in range(B):
+                    runner.run([StepEntry(r, rng.integers(0, V, CTX - steps - 8).tolist(), [])])
+                feed = rng.integers(0, V, (steps + 8, B))
+                for i in range(8):
+                    runner.run([StepEntry(r, [int(feed[i, r])], [0]) for r in range(B)])
+                marks = [ev() for _ in range(steps + 1)]
+                torch.cuda.synchronize()
+                marks[0].record()
+                for i in range(steps):
+                    runner.run([StepEntry(r, [int(feed[8 + i, r])], [0]) for r in range(B)])
+                    marks[i + 1].record()
+                torch.cuda.synchronize()
+                each = sorted(marks[i].elapsed_time(marks[i + 1]) for i in range(steps))
+                for r in range(B):
+                    runner.end(r)
+                rec[arch].update({"decode_b8_ctx2048_ms": round(each[len(each) // 2], 4),
+                                  "decode_tok_s": round(B / each[len(each) // 2] * 1e3),
+                                  "graph_replays": runner.graphs.replays,
+                                  "kernels_per_decode_step": runner.graphs.launches_replayed(B)})
+            if engine.ops.tc is not None:
+                engine.ops.tc.check_errors()
+        if args.only:
+            out["sizes"][name] = rec
+            continue
+        # ------------------------------------------------------------ kernel beside like kernel
+        ops = engines["fosovik"].ops
+        bf = torch.bfloat16
+        H, Hkv, hd, W, ps = z["heads"], z["kv_heads"], z["dim"], z["width"], 32
+        ctx = SimpleNamespace(ws=Workspace(dev), step_cache={})
+        ws, kern = ctx.ws, {}
+        for label, nreq, q_len, kv_len in (("prefill_2048", 1, T, T), ("decode_b8_ctx2048", B, 1, CTX)):
+            pages, n = (kv_len + ps - 1) // ps, nreq * q_len
+            bt = torch.arange(nreq * pages, dtype=torch.int32, device=dev).view(nreq, pages)
+            cu = torch.arange(nreq + 1, dtype=torch.int32, device=dev) * q_len
+            kvl = torch.full((nreq,), kv_len, dtype=torch.int32, device=dev)
+            req = torch.arange(nreq, dtype=torch.int32, device=dev).repeat_interleave(q_len)
+            pos = (torch.arange(q_len, dtype=torch.int32, device=dev) + (kv_len - q_len)).repeat(nreq)
+            ctx.batch = SimpleNamespace(cu_q=cu, token_req=req, positions=pos, kv_lens=kvl, num_requests=nreq, max_q_len=q_len,
+                                        min_q_len=q_len, slots=torch.arange(nreq, dtype=torch.int32, device=dev))
+            # attention with learned sinks, beside Murilorn's capped one with a sink over the same keys
+            q = torch.randn(n, H, hd, device=dev).to(bf)
+            kp, vp = (torch.randn(nreq * pages, Hkv, ps, hd, device=dev).to(bf) for _ in range(2))
+            o = torch.empty(n, H * hd, dtype=bf, device=dev)
+            sinks = torch.randn(H, device=dev)
+            keys = nreq * sum(range(kv_len - q_len + 1, kv_len + 1))
+            cost = (4.0 * H * hd * keys, 2.0 * (2 * nreq * kv_len * Hkv * hd + q.numel() + o.numel()))
+            args_a = (q, kp, vp, bt, cu, kvl, req, o, hd ** -0.5, 0, ps, nreq, q_len, kv_len)
+            kern[f"sink_attention_{label}"] = roof(timed(lambda: ops.paged_attention(*args_a, ws=ws, min_q_len=q_len, sink_values=sinks)), *cost)
+            kern[f"murilorn_capped_sink_attention_{label}"] = roof(
+                timed(lambda: ops.paged_attention(*args_a, ws=ws, min_q_len=q_len, softcap=30.0, sink=True)), *cost)
+            # the projected row into queries and pages: normed and grown here, biased there
+            row, bias = torch.randn(n, (H + 2 * Hkv) * hd, device=dev), torch.zeros((H + 2 * Hkv) * hd, device=dev)
+            qw, kw = torch.ones(H, hd, device=dev), torch.ones(hd, device=dev)
+            moved = 4.0 * row.numel() + 2.0 * row.numel()
+            kern[f"norm_grow_store_{label}"] = roof(timed(lambda: ops.qk_norm_rope_append(
+                row, (0, H * hd, (H + Hkv) * hd), q, kp, vp, pos, req, bt, H, Hkv, hd, hd, qw, kw, 1e-5, None, ps, query_growth=(0.1, 1024))), 0, moved)
+            kern[f"murilorn_bias_store_{label}"] = roof(
+                timed(lambda: ops.qkv_bias_append(row, bias, q, kp, vp, pos, req, bt, H, Hkv, hd, hd, ps)), 0, moved)
+            # the recurrences, everything between the projections: bytes are the rows in and out and the state
+            SH, SP, SN, SG, taps = z["s_heads"], z["s_vdim"], z["s_state"], z["s_groups"], z["taps"]
+            inner, C = SH * SP, SH * SP + 2 * SG * SN
+            proj = torch.randn(n, 2 * inner + 2 * SG * SN + SH, device=dev)
+            vec = lambda m, s=1.0: torch.randn(m, device=dev) * s
+            cw, cb, rate, dtb, skip, nw = vec(C * taps, 0.4).view(C, taps), vec(C, 0.1), torch.rand(SH, device=dev) * 8, vec(SH), vec(SH), vec(inner)
+            st, so = torch.zeros(nreq, inner * SN + (taps - 1) * C, device=dev), torch.empty(n, inner, dtype=bf, device=dev)
+            ms = timed(lambda: ops.state_space(ctx, proj, (0, inner, inner + C), cw, cb, rate, dtb, skip, nw, z["s_parts"], 1e-5, st, SH, SG, SN,
+                                               SP, so))
+            kern[f"state_space_{label}"] = roof(ms, 0, 4.0 * proj.numel() + 2.0 * so.numel() + 2 * 4.0 * st.numel())
+            dH, dG, dd, dv = z["d_heads"], z["d_kv_heads"], z["d_dim"], z["d_vdim"]
+            DC = 2 * dG * dd + dH * dv
+            conv_w, a_log, dnw = torch.randn(DC, taps, device=dev) * 0.3, vec(dH, 0.3), torch.ones(dv, device=dev)
+            dstate = torch.zeros(nreq, dH * dd * dv + (taps - 1) * DC, device=dev)
+            dproj, second = torch.randn(n, DC + dH, device=dev), torch.randn(n, dH * dd + dH * dv, device=dev)
+            ddt, do = vec(dH * dd), torch.empty(n, dH * dv, dtype=bf, device=dev)
+            ms = timed(lambda: ops.delta_rule(ctx, dproj, second, conv_w, a_log, ddt, dnw, 1e-5, dstate, dH, dG, dd, dv, taps, do))
+            kern[f"murilorn_channel_delta_rule_{label}"] = roof(ms, 0, 4.0 * (dproj.numel() + second.numel()) + 2.0 * do.numel()
+                                                                + 2 * 4.0 * dstate.numel())
+            del q, kp, vp, o, row, proj, so, dproj, second, do
+        # feed-forwards: experts of two products here, of three there; the clamped dense one beside Llama's
+        FF, E, top, EF = z["ff"], z["experts"], z["top"], z["expert_ff"]
+        mat = lambda *s: (torch.randn(*s, device=dev) * 0.02).to(bf)
+        for label, M in (("2048_tokens", T), ("8_tokens", B)):
+            h, x = torch.randn(M, W, device=dev).to(bf), torch.zeros(M, W, device=dev)
+            ids = torch.stack([torch.randperm(E, device=dev)[:top] for _ in range(M)]).to(torch.int32)
+            wts = torch.rand(M, top, device=dev)
+            up, down = mat(E, EF, W), mat(E, W, EF)
+            gu = ops.pack_expert_gate_up([mat(EF, W) for _ in range(E)], [mat(EF, W) for _ in range(E)])
+            used = E if M > 8 else len(torch.unique(ids))
+            ms = timed(lambda: ops.routed_feed_forward(ctx, h, up, down, ids, wts, x, "gelu", 0.0, gated=False))
+            kern[f"gelu_experts_{label}"] = roof(ms, 2.0 * M * top * 2 * EF * W, 2.0 * used * 2 * EF * W)
+            ms = timed(lambda: ops.routed_feed_forward(ctx, h, gu, down, ids, wts, x, "silu", 0.0))
+            kern[f"murilorn_gated_experts_{label}"] = roof(ms, 2.0 * M * top * 3 * EF * W, 2.0 * used * 3 * EF * W)
+            del up, down, gu
+            g, dwn, act = ops.pack_gate_up(mat(FF, W), mat(FF, W)), mat(W, FF), torch.empty(M, FF, dtype=bf, device=dev)
+
+            def dense(kind, limit):
+                ops.linear_gated(ctx, h, g, act, kind, limit)
+                ops.linear(act, dwn, x, accumulate=True)
+
+            cost = (2.0 * M * 3 * FF * W, 2.0 * 3 * FF * W)
+            kern[f"clamped_feed_forward_{label}"] = roof(timed(lambda: dense("clamped_swish", 7.0)), *cost)
+            kern[f"llama_silu_feed_forward_{label}"] = roof(timed(lambda: dense("silu", 0.0)), *cost)
+            del g, dwn, act
+        wv, xr, hb = torch.ones(W, device=dev), torch.randn(T, W, device=dev), torch.empty(T, W, dtype=bf, device=dev)
+        kern["dynamic_tanh_2048_tokens"] = roof(timed(lambda: ops.dynamic_tanh(xr, 0.5, wv, wv, hb)), 0, 6.0 * T * W)
+        kern["llama_rms_norm_2048_tokens"] = roof(timed(lambda: ops.rmsnorm(xr, wv, 1e-5, hb)), 0, 6.0 * T * W)
+        rec["kernels"] = kern
+        rec["config"] = {k: v for k, v in z.items()}
+        out["sizes"][name] = rec
+        del engines
+        torch.cuda.empty_cache()
+    return out
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1373,8 +1587,8 @@ def main() -> int:
     ap.add_argument("--context", type=int, default=0, help="context reached with --only decode (default: the shape's); keys with --only attention")
     ap.add_argument("--layers", type=int, default=0,
                     help="fewer layers than the configuration has (reported beside the full number)")
-    ap.add_argument("--design", choices=["kavenex", "murilorn", "luvapel", "midulorn"],
-                    help="instead of the default workload: this design beside the Llama decoder (luvapel and midulorn: "
+    ap.add_argument("--design", choices=["kavenex", "murilorn", "luvapel", "midulorn", "fosovik"],
+                    help="instead of the default workload: this design beside the Llama decoder (luvapel, midulorn and fosovik: "
                          "beside Murilorn, the closest of the engine's models) at equal sizes")
     ap.add_argument("--size", default="", help="with --design: which of its sizes (2k, 4k; default both)")
     args = ap.parse_args()
@@ -1393,7 +1607,7 @@ def main() -> int:
         return 2
     if args.design:
         run = {"murilorn": run_design_murilorn, "luvapel": run_design_luvapel, "kavenex": run_design,
-               "midulorn": run_design_midulorn}[args.design]
+               "midulorn": run_design_midulorn, "fosovik": run_design_fosovik}[args.design]
         print(json.dumps(run(args)))
         return 0
     print(json.dumps(run_ours(args)))
