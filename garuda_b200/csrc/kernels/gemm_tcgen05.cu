@@ -231,6 +231,20 @@ __device__ __forceinline__ float gate_fast(const EpilogueArgs& ra, float g, floa
   return g * __frcp_rn(1.0f + __expf(-1.702f * g)) * (u + 1.0f);
 }
 
+// The exact gelu, z Phi(z). The complementary error function by formula 7.1.26 of Abramowitz and Stegun's "Handbook of
+// Mathematical Functions": erfc(x) = (a1 t + ... + a5 t^5) exp(-x^2), t = 1 / (1 + p x), x >= 0, absolute error below
+// 1.5e-7, which is far below the rounding of the bfloat16 result. Without a branch, two special-function instructions.
+__device__ __forceinline__ float gelu_fast(float z) {
+  const float x = fabsf(z) * 0.7071067811865476f;
+  const float t = __fdividef(1.0f, fmaf(0.3275911f, x, 1.0f));
+  float q = fmaf(t, 1.061405429f, -1.453152027f);
+  q = fmaf(t, q, 1.421413741f);
+  q = fmaf(t, q, -0.284496736f);
+  q = fmaf(t, q, 0.254829592f);
+  const float tail = 0.5f * q * t * __expf(-x * x);        // Phi(-|z|)
+  return z * (z > 0.f ? 1.0f - tail : tail);
+}
+
 // The storing epilogue's activation of one value (EPI_STORE | EPI_GENERAL), uniform over the launch.
 __device__ __forceinline__ float store_act_fast(const EpilogueArgs& ra, float z) {
   if (ra.gate_act == STORE_RELU2) {
@@ -241,8 +255,27 @@ __device__ __forceinline__ float store_act_fast(const EpilogueArgs& ra, float z)
     const float half = 0.5f * z;
     return z > 0.f ? fmaf(ra.gate_limit * z, z, half) : fmaf(ra.act_second, __expf(z) - 1.0f - z, half);
   }
-  if (ra.gate_act == STORE_GELU) return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
+  if (ra.gate_act == STORE_GELU) return gelu_fast(z);
   return 1.0f - 2.0f * __frcp_rn(__expf(2.0f * z) + 1.0f);
+}
+
+// The same for a whole tile's 32 columns of a thread: the kind is looked at once, not per value.
+__device__ __forceinline__ void store_act_32(const EpilogueArgs& ra, uint32_t (&r)[32]) {
+#define GB_EACH(EXPR)                                  \
+  _Pragma("unroll") for (int j = 0; j < 32; ++j) {     \
+    const float z = __uint_as_float(r[j]);             \
+    r[j] = __float_as_uint(EXPR);                      \
+  }
+  if (ra.gate_act == STORE_GELU) {
+    GB_EACH(gelu_fast(z))
+  } else if (ra.gate_act == STORE_RELU2) {
+    GB_EACH(fmaxf(z, 0.f) * fmaxf(z, 0.f))
+  } else if (ra.gate_act == STORE_XIELU) {
+    GB_EACH(z > 0.f ? fmaf(ra.gate_limit * z, z, 0.5f * z) : fmaf(ra.act_second, __expf(z) - 1.0f - z, 0.5f * z))
+  } else {
+    GB_EACH(1.0f - 2.0f * __frcp_rn(__expf(2.0f * z) + 1.0f))
+  }
+#undef GB_EACH
 }
 
 // Sums each of sixteen values over the lanes of a warp with sixteen shuffles: at every step a
@@ -791,7 +824,8 @@ __device__ __forceinline__ void epilogue_tile(uint32_t taddr, int row, int n0, O
       for (int rr = 0; rr < 32; ++rr) old_cur[ACC ? rr : 0] = first[ACC ? rr : 0];
     }
     constexpr int BLOCKS = BN / 32 / (epilogue_warps(EPI) / 4);     // blocks of 32 columns per warp
-    constexpr int UNROLL = ACC ? 1 : BLOCKS;                       // the folded norm's work needs the registers
+    constexpr bool ACT = (EPI & 7) == EPI_STORE && (EPI & EPI_GENERAL) != 0;
+    constexpr int UNROLL = ACC || ACT ? 1 : BLOCKS;                // the folded norm's work needs the registers, an activation the instruction cache
 #pragma unroll UNROLL
     for (int k = 0; k < BLOCKS; ++k) {
       const int c = c_begin + 32 * k;
@@ -800,6 +834,7 @@ __device__ __forceinline__ void epilogue_tile(uint32_t taddr, int row, int n0, O
       tmem_ld_32(taddr + c, r);
       if (ACC && k > 0) fetch(old_cur, c);
       tmem_ld_wait();
+      if (ACT) store_act_32(ra, r);
 #pragma unroll
       for (int j = 0; j < 32; ++j) turn[lane * 33 + j] = __uint_as_float(r[j]);
       __syncwarp();
@@ -807,7 +842,6 @@ __device__ __forceinline__ void epilogue_tile(uint32_t taddr, int row, int n0, O
 #pragma unroll
       for (int rr = 0; rr < 32; ++rr) {
         float v = turn[rr * 33 + lane];
-        if ((EPI & 7) == EPI_STORE && (EPI & EPI_GENERAL)) v = store_act_fast(ra, v);
         if (ACC) v = (EPI & EPI_GENERAL) ? fmaf(ra.alpha, v, old_cur[ACC ? rr : 0]) : v + old_cur[ACC ? rr : 0];
         if (rr < rows_valid) store_value<OT>(gbase + (size_t)rr * ldo + c, v);
         if (EMIT) {
