@@ -226,7 +226,8 @@ __global__ void rope_inplace_kernel(float* __restrict__ x, int row_stride, int h
 enum GbGateAct : int { GB_ACT_SILU = 0, GB_ACT_GELU_TANH = 1, GB_ACT_CLAMPED_SWISH = 2 };
 
 __device__ __forceinline__ float gelu_tanh(float z) {
-  return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  // (1 + tanh v) / 2 is the sigmoid of 2 v, which loses nothing where tanh is close to -1
+  return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
 }
 
 __device__ __forceinline__ float gate_act(int kind, float limit, float g, float u) {

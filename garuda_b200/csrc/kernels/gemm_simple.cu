@@ -3,9 +3,8 @@
 // beside the tensor-core kernels. garuda/src/simd/mod.rs:96-129 (`matmul`: each
 // output is the dot of one matrix row with one input vector, :13-16).
 //
-// Every output element is one thread's sum over k = 0..K-1, sixteen terms summed by themselves and the
-// sixteens added up in order (rounding grows with 16 + K / 16 additions, not with K), whatever M is, so a
-// token's result does not depend on the rest of the batch.
+// Every output element is one thread's sum over k = 0..K-1 in that order,
+// whatever M is, so a token's result does not depend on the rest of the batch.
 #include "common.cuh"
 
 namespace {
@@ -38,11 +37,6 @@ gemm_simple_kernel(const IT* __restrict__ a, const IT* __restrict__ w, OT* __res
       Ws[c][r] = (gn < N && gk < K) ? gb::to_float<IT>(w[(size_t)gn * K + gk]) : 0.f;
     }
     __syncthreads();
-    float part[TM][TN];
-#pragma unroll
-    for (int i = 0; i < TM; ++i)
-#pragma unroll
-      for (int j = 0; j < TN; ++j) part[i][j] = 0.f;
 #pragma unroll
     for (int k = 0; k < BK; ++k) {
       float av[TM], wv[TN];
@@ -53,12 +47,8 @@ gemm_simple_kernel(const IT* __restrict__ a, const IT* __restrict__ w, OT* __res
 #pragma unroll
       for (int i = 0; i < TM; ++i)
 #pragma unroll
-        for (int j = 0; j < TN; ++j) part[i][j] = fmaf(av[i], wv[j], part[i][j]);
+        for (int j = 0; j < TN; ++j) acc[i][j] = fmaf(av[i], wv[j], acc[i][j]);
     }
-#pragma unroll
-    for (int i = 0; i < TM; ++i)
-#pragma unroll
-      for (int j = 0; j < TN; ++j) acc[i][j] += part[i][j];
     __syncthreads();
   }
 #pragma unroll

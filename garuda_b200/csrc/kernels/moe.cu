@@ -82,7 +82,7 @@ route_topk_kernel(const HT* __restrict__ h, const WT* __restrict__ w, const floa
 }
 
 __device__ __forceinline__ float gate_act(int kind, float limit, float g, float u) {
-  if (kind == 1) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+  if (kind == 1) return g / (1.0f + expf(-1.5957691216057308f * (g + 0.044715f * g * g * g))) * u;      // (1 + tanh v) / 2 is the sigmoid of 2 v
   if (kind == 2) {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
@@ -98,7 +98,7 @@ __device__ __forceinline__ float plain_act(int kind, float z) {
     case 1: return z / (1.0f + expf(-z));
     case 2: return fmaxf(z, 0.f) * fmaxf(z, 0.f);
     case 3: return tanhf(z);
-    default: return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
+    default: return 0.5f * z * erfcf(z * -0.7071067811865476f);
   }
 }
 

@@ -113,7 +113,7 @@ __device__ __forceinline__ float act(float z, int kind) {
     case ACT_SIGMOID: return sigmoidf_(z);
     case ACT_SILU: return z * sigmoidf_(z);
     case ACT_RELU2: { const float r = fmaxf(z, 0.f); return r * r; }
-    case ACT_GELU: return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f));
+    case ACT_GELU: return 0.5f * z * erfcf(z * -0.7071067811865476f);
     default: return tanhf(z);
   }
 }
