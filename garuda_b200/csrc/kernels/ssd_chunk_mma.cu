@@ -119,15 +119,19 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ act, int C, const float* __re
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  // warp 0: a chunk's running sums of log decays (lane l has tokens 2 l and 2 l + 1; beyond the end: dt 0, decay one)
-  auto decays = [&](int chunk, int st) {
+  // (Tokens beyond a request's last are zeros in every operand: a short chunk runs the same instructions, which the
+  // compiler may then interleave freely.) The last warp: a chunk's running sums of log decays (lane l has tokens 2 l and 2 l + 1; beyond the end: dt 0,
+  // decay one), from values asked for a chunk ahead.
+  float d[2], a[2];
+  auto ask_decays = [&](int chunk) {
     const int t = t0 + chunk * Q + 2 * lane;
-    float d[2], a[2];
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       d[e] = t + e < t1 ? step[(size_t)(t + e) * 2 * H + h] : 0.f;
       a[e] = t + e < t1 ? step[(size_t)(t + e) * 2 * H + H + h] : 0.f;
     }
+  };
+  auto decays = [&](int st) {
     float run = a[0] + a[1];
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
@@ -163,22 +167,22 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ act, int C, const float* __re
   const float dskip = skip[h];
   const int chunks = (t1 - t0 + Q - 1) / Q;
   load(0, 0);
-  if (warp == 0) decays(0, 0);
+  if (warp == WARPS - 1) {
+    ask_decays(0);
+    decays(0);
+    ask_decays(1);
+  }
   for (int ck = 0; ck < chunks; ++ck) {
     const int st = ck & 1;
     const Stage& s = sm.stage[st];
-    const int blocks = (min(Q, t1 - t0 - ck * Q) + 15) / 16;     // blocks of 16 tokens that hold any
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();           // this chunk has landed; everyone is done with the chunk in front (its buffers, y's shares)
-    if (ck + 1 < chunks) {
-      load(ck + 1, st ^ 1);
-      if (warp == 0) decays(ck + 1, st ^ 1);
-    }
+    if (ck + 1 < chunks) load(ck + 1, st ^ 1);
     // ---- M, its lower triangle
 #pragma unroll
     for (int k = 0; k < 2; ++k) {
       int ib, jb;
-      if (!m_block(warp, k, ib, jb) || ib >= blocks) continue;
+      if (!m_block(warp, k, ib, jb)) continue;
       float acc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll
       for (int kk = 0; kk < NT; ++kk) {
@@ -226,7 +230,6 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ act, int C, const float* __re
         }
 #pragma unroll
       for (int ib = 0; ib < Q / 16; ++ib) {
-        if (ib >= blocks) break;
         uint32_t b[4];
         ldmatrix_x4(b, &s.c[ib * 16 + (lane & 7) + (lane >> 4) * 8][nb * 16 + ((lane >> 3) & 1) * 8]);
 #pragma unroll
@@ -252,7 +255,6 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ act, int C, const float* __re
           for (int e = 0; e < 4; ++e) S[m][half][e] *= whole;
 #pragma unroll
       for (int jb = 0; jb < Q / 16; ++jb) {
-        if (jb >= blocks) break;
         uint32_t xt[4], a[SPLIT][4];
         ldmatrix_x4_trans(xt, &s.x[jb * 16 + (lane & 7) + (lane >> 4) * 8][pr * 16 + ((lane >> 3) & 1) * 8]);
 #pragma unroll
@@ -277,17 +279,21 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ act, int C, const float* __re
         }
       }
     }
+    if (ck + 1 < chunks && warp == WARPS - 1) {
+      decays(st ^ 1);
+      ask_decays(ck + 2);
+    }
     __syncthreads();           // M is whole
     // ---- the chunk's own part of y^T: x^T M^T over this warp's token blocks
 #pragma unroll
     for (int k = 0; k < (Q / 16 + KS - 1) / KS; ++k) {
       const int jb = (k & 1) ? (k + 1) * KS - 1 - kh : k * KS + kh;       // blocks early and late in turn: they differ in length
-      if (jb >= blocks) continue;
+      if (jb >= Q / 16) continue;
       uint32_t xt[4];
       ldmatrix_x4_trans(xt, &s.x[jb * 16 + (lane & 7) + (lane >> 4) * 8][pr * 16 + ((lane >> 3) & 1) * 8]);
 #pragma unroll
       for (int ib = 0; ib < Q / 16; ++ib) {
-        if (ib < jb || ib >= blocks) continue;
+        if (ib < jb) continue;
 #pragma unroll
         for (int q = SPLIT - 1; q >= 0; --q) {
           uint32_t b[4];
