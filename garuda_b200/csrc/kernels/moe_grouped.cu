@@ -226,10 +226,17 @@ grouped_gemm_kernel(const __nv_bfloat16* __restrict__ a, int lda, long long a_gr
       }
 }
 
+// A norm without statistics that the next layer starts with: out = tanh(alpha x) w + b of the new x, bfloat16 (out null: none).
+struct TanhNorm {
+  __nv_bfloat16* out;
+  const float *w, *b;
+  float alpha;
+};
+
 // x[t][n] += alpha * sum_j weights[t][j] * y[pair_row[t * top + j]][n], j in the router's order; weights null: all one
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ y, const int32_t* __restrict__ pair_row, const float* __restrict__ weights,
-                   float* __restrict__ x, int top, int N, float alpha) {
+                   float* __restrict__ x, int top, int N, float alpha, const TanhNorm norm) {
   const int t = blockIdx.x;
   for (int n = threadIdx.x; n < N; n += blockDim.x) {
     float total = 0.f;
@@ -237,7 +244,9 @@ moe_combine_kernel(const float* __restrict__ y, const int32_t* __restrict__ pair
       const int row = pair_row[(size_t)t * top + j];
       if (row >= 0) total = fmaf(weights ? weights[(size_t)t * top + j] : 1.0f, y[(size_t)row * N + n], total);
     }
-    x[(size_t)t * N + n] = fmaf(alpha, total, x[(size_t)t * N + n]);
+    const float v = fmaf(alpha, total, x[(size_t)t * N + n]);
+    x[(size_t)t * N + n] = v;
+    if (norm.out != nullptr) norm.out[(size_t)t * N + n] = __float2bfloat16_rn(fmaf(tanhf(norm.alpha * v), norm.w[n], norm.b[n]));
   }
 }
 
@@ -272,7 +281,7 @@ GB_EXPORT long long gb_moe_grouped_index_words(long long R, int E) {
 GB_EXPORT int gb_moe_grouped(const void* h, const void* w_gate_up, const void* w_down, const int32_t* ids,
                              const float* weights, float* x, int T, int top, int E, int F, int K, int N, int kind,
                              float limit, float alpha, int layout, int scale_input, int32_t* index, void* act, float* y,
-                             cudaStream_t stream) {
+                             void* norm_out, const float* norm_w, const float* norm_b, float norm_alpha, cudaStream_t stream) {
   if (T <= 0) return GB_OK;
   if (K % 8 || F % 8) return gb::fail(GB_UNSUPPORTED, "moe_grouped: widths %d and %d must be multiples of 8", K, F);
   if (E < 1 || (size_t)E * 2 * sizeof(int32_t) > 40 * 1024) return gb::fail(GB_UNSUPPORTED, "moe_grouped: %d experts", E);
@@ -325,7 +334,8 @@ GB_EXPORT int gb_moe_grouped(const void* h, const void* w_gate_up, const void* w
     rc = launch_grouped<1, 4, 1, 1, PLAIN, float>(grid_n, stream, "moe_down_grouped", ac, F, zero, none, 1, wd, d_group, y, N,
                                                  zero, N, F, te, t0, tr, nt, 0, 0, 0.f, 0, no_scale);
   if (rc != GB_OK) return rc;
-  moe_combine_kernel<<<T, 256, 0, stream>>>(y, pair_row, out_weights, x, top, N, alpha);
+  moe_combine_kernel<<<T, 256, 0, stream>>>(y, pair_row, out_weights, x, top, N, alpha,
+                                            TanhNorm{(__nv_bfloat16*)norm_out, norm_w, norm_b, norm_alpha});
   return gb::check_launch("moe_combine");
 }
 
@@ -421,11 +431,14 @@ GB_EXPORT int gb_moe_padded_prepare(const void* h, const int32_t* ids, int T, in
   return gb::check_launch("moe_gather_rows");
 }
 
-// x[t] += alpha * sum_j weights[t][j] * y[pair_row[t * top + j]], j in the router's order
+// x[t] += alpha * sum_j weights[t][j] * y[pair_row[t * top + j]], j in the router's order; norm_out (or null): also
+// tanh(norm_alpha x) norm_w + norm_b of the new x, bfloat16 (likewise for gb_moe_grouped)
 GB_EXPORT int gb_moe_combine(const float* y, const int32_t* pair_row, const float* weights, float* x, int T, int top,
-                             int N, float alpha, cudaStream_t stream) {
+                             int N, float alpha, void* norm_out, const float* norm_w, const float* norm_b, float norm_alpha,
+                             cudaStream_t stream) {
   if (T <= 0) return GB_OK;
-  moe_combine_kernel<<<T, 256, 0, stream>>>(y, pair_row, weights, x, top, N, alpha);
+  moe_combine_kernel<<<T, 256, 0, stream>>>(y, pair_row, weights, x, top, N, alpha,
+                                            TanhNorm{(__nv_bfloat16*)norm_out, norm_w, norm_b, norm_alpha});
   return gb::check_launch("moe_combine");
 }
 

@@ -285,10 +285,11 @@ class CudaOps:
                           c_void_p],
             "gb_moe_down": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                             c_float, c_void_p],
-            "gb_moe_grouped": [c_void_p] * 6 + [c_int] * 7 + [c_float, c_float, c_int, c_int] + [c_void_p] * 4,
+            "gb_moe_grouped": [c_void_p] * 6 + [c_int] * 7 + [c_float, c_float, c_int, c_int] + [c_void_p] * 6 + [c_float, c_void_p],
             "gb_moe_padded_prepare": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
                                       c_void_p, c_void_p],
-            "gb_moe_combine": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
+            "gb_moe_combine": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p,
+                               c_float, c_void_p],
             "gb_grouped_gemm": [c_void_p, c_int, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_longlong,
                                 c_int, c_int, c_int, c_int, c_void_p],
             "gb_latent_query_prepare": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
@@ -785,14 +786,20 @@ class CudaOps:
             return packed
         return torch.stack([torch.cat([g, u], dim=0) for g, u in zip(gates, ups)]).contiguous()
 
+    #: the experts' last pass may also compute a norm without statistics of the residual it writes (``then``)
+    fuses_tanh_norms = True
+
     #: (token, choice) pairs from which the routed experts run on the tcgen05 grouped product
     GROUPED_TC_PAIRS = 1024
 
     def routed_feed_forward(self, ctx, h, w_gate_up, w_down, ids, weights, x, kind: str, limit: float,
-                            alpha: float = 1.0, scale_input: bool = False, gated: bool = True):
+                            alpha: float = 1.0, scale_input: bool = False, gated: bool = True, then=None):
         """``x[t] += alpha * sum_j weights[t, j] * expert_{ids[t, j]}(h[t])`` with the experts'
         weights stacked: ``w_gate_up`` from ``pack_expert_gate_up``, ``w_down [E, N, F]``. Without ``gated``:
         ``w_gate_up`` is ``[E, F, K]``, the up rows alone, and ``kind`` an activation of one value.
+        ``then = (alpha, weight, bias, out)``: the pass that writes ``x`` also writes ``tanh(alpha x) weight + bias``
+        (32-bit vectors) into ``out`` (bfloat16 ``[T, N]``), where the tensor-core kernels take the sizes; returns
+        whether it did.
         ``scale_input``: the weight multiplies what goes into the expert instead,
         ``sum_j expert(weights[t, j] * h[t])``."""
         T, top = ids.shape
@@ -801,8 +808,9 @@ class CudaOps:
         packed = getattr(w_gate_up, "gb_group", 0) == 64
         grouped = packed if gated else (self.tc is not None and h.dtype == torch.bfloat16 and K % 8 == 0 and F % 8 == 0 and E <= 4096)
         if grouped and T * top >= self.GROUPED_TC_PAIRS and self._routed_tcgen05(ctx, h, w_gate_up, w_down, ids, weights,
-                                                                                x, kind, limit, alpha, scale_input, gated):
-            return
+                                                                                x, kind, limit, alpha, scale_input, gated, then):
+            return then is not None
+        norm = self._then_norm(then, T, N)
         if grouped:
             # on the tensor cores: pairs sorted by expert on the device, two grouped products, a weighted sum
             self._on_device(h, w_gate_up, w_down, ids, weights, x)
@@ -820,17 +828,27 @@ class CudaOps:
                 h.data_ptr(), w_gate_up.data_ptr(), w_down.data_ptr(), ids.data_ptr(), weights.data_ptr(), x.data_ptr(),
                 T, top, E, F, K, N, self.GATE_ACTS[kind] if gated else self.UNARY_ACTS[kind], float(limit), float(alpha),
                 1 if gated else 2, int(scale_input), index.data_ptr(),
-                act.data_ptr(), y.data_ptr(), self._stream()), "moe_grouped", 4)
-            return
+                act.data_ptr(), y.data_ptr(), *norm, self._stream()), "moe_grouped", 4)
+            return then is not None
         act = ctx.ws.get("expert_act", (T, top, F), h.dtype)
         if gated:
             self.moe_gate_up(h, w_gate_up, ids, act, kind, limit, weights if scale_input else None)
         else:
             self.moe_up(h, w_gate_up, ids, act, kind, weights if scale_input else None)
         self.moe_down(act, w_down, ids, None if scale_input else weights, x, alpha)
+        return False
+
+    def _then_norm(self, then, rows, width):
+        if then is None:
+            return (None, None, None, 0.0)
+        alpha, w, b, out = then
+        self._on_device(w, b, out)
+        _need(out.dtype == torch.bfloat16 and out.is_contiguous() and tuple(out.shape) == (rows, width)
+              and all(v.dtype == torch.float32 and v.is_contiguous() and v.numel() == width for v in (w, b)), "then: out, weight, bias")
+        return (out.data_ptr(), w.data_ptr(), b.data_ptr(), float(alpha))
 
     def _routed_tcgen05(self, ctx, h, w_gate_up, w_down, ids, weights, x, kind, limit, alpha, scale_input=False,
-                        gated=True) -> bool:
+                        gated=True, then=None) -> bool:
         """Many pairs: sorted by expert into blocks of 128 rows (padding rows zero), then the two
         products on the tcgen05 many-token kernel with each block's expert read from a list."""
         T, top = ids.shape
@@ -865,7 +883,7 @@ class CudaOps:
             tc.grouped(a, w_gate_up, act, F, E, block_gu, 0, gate_act=tc.STORE_ACTS[kind])
         tc.grouped(act, w_down, y, N, E, block_dn, 0)
         self._check(L, L.gb_moe_combine(y.data_ptr(), index.data_ptr(), None if scale_input else weights.data_ptr(), x.data_ptr(), T, top, N,
-                                        float(alpha), self._stream()), "moe_combine")
+                                        float(alpha), *self._then_norm(then, T, N), self._stream()), "moe_combine")
         return True
 
     # ------------------------------------------------------------------ attention over a cached latent

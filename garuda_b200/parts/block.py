@@ -16,6 +16,7 @@ from typing import Optional, Tuple
 
 import torch
 
+from .norm import DynamicTanh
 from .base import PartSpec, SublayerGate, TensorSpec, build_part, register_block, register_gate
 
 
@@ -411,19 +412,35 @@ class ParallelBlock:
     def graph_safe(self):
         return all(part.graph_safe for part, _ in self.parts())
 
+    def takes_pending_norm(self, ops):
+        """A layer in front whose last pass over the residual can compute this layer's norm (one without
+        statistics: a function of each value) writes it."""
+        if getattr(ops, "fuses_tanh_norms", False) and isinstance(self.norm, DynamicTanh):
+            return self.norm
+        return None
+
     _run_scaled = PreNormBlock._run
 
-    def _run(self, ctx, part, x, h, *cache):
+    def _run(self, ctx, part, x, h, *cache, **kw):
         if self.mult != 1.0:
             return self._run_scaled(ctx, part, x, h, *cache)
-        y = part.forward(ctx, h, *cache, residual=x)
+        y = part.forward(ctx, h, *cache, residual=x, **kw)
         if y is not None:
             ctx.ops.residual_add(x, y)
 
-    def forward(self, ctx, x, cache):
+    def forward(self, ctx, x, cache, pending=None, next_norm=None):
+        """``pending``: this layer's normed input, written by the layer in front. ``next_norm``: the norm that the
+        next layer starts with, if it takes such a result. Returns the next layer's normed input, or None."""
+        h = pending if pending is not None else self.norm.forward(ctx, x)
+        ff = self.feed_forward
         ctx.pending_norm = None
-        h = self.norm.forward(ctx, x)
         self._run(ctx, self.mixer, x, h, cache)
-        if self.feed_forward is not None:
-            self._run(ctx, self.feed_forward, x, h)
-        return None
+        if ff is None:
+            return None
+        ctx.pending_norm = None
+        kw = {}
+        if self.mult == 1.0 and isinstance(next_norm, DynamicTanh) and ctx.dtype == torch.bfloat16 and getattr(ff, "emits_tanh_norm", False):
+            kw["emit_norm"] = next_norm
+        self._run(ctx, ff, x, h, **kw)
+        out, ctx.pending_norm = ctx.pending_norm, None
+        return out

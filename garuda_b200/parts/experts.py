@@ -86,7 +86,12 @@ class RoutedExperts(FeedForward):
             self.w_shared_gate_up = ops.pack_gate_up(tensors["shared.gate"], tensors["shared.up"])
             self.w_shared_down = tensors["shared.down"].contiguous()
 
-    def forward(self, ctx, h, residual=None, alpha: float = 1.0):
+    @property
+    def emits_tanh_norm(self):
+        """Whether ``forward`` takes ``emit_norm``, a ``DynamicTanh`` of the residual that this part is the last to write."""
+        return not self.shared_inner
+
+    def forward(self, ctx, h, residual=None, alpha: float = 1.0, emit_norm=None):
         ops, ws = self.ops, ctx.ws
         T = h.shape[0]
         target = residual
@@ -103,8 +108,14 @@ class RoutedExperts(FeedForward):
         else:
             ops.route_topk(h, self.w_router, self.b_router, self.top, ids, weights, score=self.router_score)
             kw = {} if self.gated else {"gated": False}
-            ops.routed_feed_forward(ctx, h, self.w_gate_up, self.w_down, ids, weights, target, self.activation,
-                                    self.limit, alpha, scale_input=self.scale_input, **kw)
+            if emit_norm is not None and residual is not None:
+                turn = ctx.step_cache["tanh_turn"] = ctx.step_cache.get("tanh_turn", 0) ^ 1       # the norm in front may still be read
+                kw["then"] = (emit_norm.alpha, emit_norm.weight, emit_norm.bias,
+                              ws.get(f"tanh_normed_{turn}", (T, self.width), torch.bfloat16))
+            emitted = ops.routed_feed_forward(ctx, h, self.w_gate_up, self.w_down, ids, weights, target, self.activation,
+                                              self.limit, alpha, scale_input=self.scale_input, **kw)
+            if emitted:
+                ctx.pending_norm = kw["then"][3]
         if self.shared_inner:
             act = ws.get("shared_act", (T, self.shared_inner), self.dtype)
             ops.linear_gated(ctx, h, self.w_shared_gate_up, act, self.activation, self.shared_limit)

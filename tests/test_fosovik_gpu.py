@@ -143,6 +143,44 @@ def test_experts_without_a_gate(both, T, E, K, F, top, N, kind):
         close(got, want, dt, f"experts {kind}")
 
 
+@pytest.mark.parametrize("T", [1, 9, 150, 700])
+def test_the_experts_last_pass_computes_the_next_norm(T):
+    """On the tensor-core paths (few pairs and many): the residual as without it, and its norm bit for bit as the norm's
+    own kernel computes it; sizes that run on the plain kernels say that they did not."""
+    from garuda_b200.kernels.ops import CudaOps
+    ops = CudaOps("cuda:0")
+    bf = torch.bfloat16
+    for E, K, F, top, N, does in ((6, 128, 64, 3, 136, True), (6, 44, 24, 3, 44, False)):
+        h, up, down = (rnd(*s, dtype=bf, scale=0.3, seed=i).cuda() for i, s in enumerate(((T, K), (E, F, K), (E, N, F))))
+        ids = torch.stack([torch.randperm(E)[:top] for _ in range(T)]).to(torch.int32).cuda()
+        wts, w, b = torch.rand(T, top).cuda(), rnd(N, seed=5).cuda(), rnd(N, seed=6).cuda()
+        x = rnd(T, N, seed=7).cuda()
+        y, out = x.clone(), torch.full((T, N), 9.0, dtype=bf, device="cuda")
+        ops.routed_feed_forward(_Ctx(), h, up, down, ids, wts, x, "gelu", 0.0, gated=False)
+        assert bool(ops.routed_feed_forward(_Ctx(), h, up, down, ids, wts, y, "gelu", 0.0, gated=False, then=(0.6, w, b, out))) == does
+        assert torch.equal(x, y)
+        if does:
+            want = torch.empty_like(out)
+            ops.dynamic_tanh(x, 0.6, w, b, want)
+            assert torch.equal(out, want)
+        else:
+            assert (out == 9.0).all()
+
+
+def test_norms_in_the_experts_last_pass_leave_the_logits_as_they_were():
+    from garuda_b200 import Engine, StepEntry
+    name = "FB"
+    toks = random_tokens(name, 60, 12)
+    e = Engine(model_dir(name, torch.bfloat16), dtype="bfloat16", context=256, kv_tokens=512, max_concurrent=2)
+    seen = []
+    for fused in (True, False):
+        e.ops.fuses_tanh_norms = fused
+        out = [e.step([StepEntry(1, toks[:40], range(40))]).cpu().clone(), e.step([StepEntry(1, toks[40:43], range(3))]).cpu().clone()]
+        e.runner.end(1)
+        seen.append(torch.cat(out))
+    assert torch.equal(seen[0], seen[1])
+
+
 @pytest.mark.parametrize("M,N,K", [(21, 77, 40), (3, 320, 160), (300, 1024, 256), (2048, 512, 128)])
 def test_exact_gelu_behind_a_product(both, M, N, K):
     ops, ref, dt = both
