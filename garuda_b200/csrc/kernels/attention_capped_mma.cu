@@ -441,7 +441,8 @@ capped_attention_kernel(const Params p) {
   }
 }
 
-// grid (Hkv, R): the shares of a decode request's keys, merged in split order; the sink joins here.
+// grid (Hkv, R, rows of a request): the shares of a decode request's keys for one row, merged in split order; the
+// sink joins here.
 __global__ void __launch_bounds__(THREADS)
 capped_attention_merge_kernel(const Params p) {
   gb::pdl_launch_dependents();
@@ -449,13 +450,15 @@ capped_attention_merge_kernel(const Params p) {
   const int kvh = blockIdx.x, r = blockIdx.y;
   const int q_begin = p.cu_q[r], q_len = p.cu_q[r + 1] - q_begin;
   if (q_len * p.g > ROWS_DECODE || q_len <= 0) return;
-  const int nrows = q_len * p.g;
+  const int row = blockIdx.z;
+  if (row >= q_len * p.g) return;
   const float* base = p.partials + ((size_t)r * p.Hkv + kvh) * p.splits * ROWS_DECODE * PR;
-  for (int idx = threadIdx.x; idx < nrows * VD; idx += THREADS) {
-    const int row = idx / VD, c = idx % VD;
+  for (int c = threadIdx.x; c < VD; c += THREADS) {
     float m = -INFINITY;
+#pragma unroll 8
     for (int s = 0; s < p.splits; ++s) m = fmaxf(m, base[((size_t)s * ROWS_DECODE + row) * PR + VD]);
     float o = 0.f, l = 0.f;
+#pragma unroll 8
     for (int s = 0; s < p.splits; ++s) {
       const float* pr = base + ((size_t)s * ROWS_DECODE + row) * PR;
       const float f = pr[VD] == -INFINITY ? 0.f : fast_exp2((pr[VD] - m) * LOG2E);
@@ -524,7 +527,7 @@ GB_EXPORT int gb_capped_attention(const void* q, const void* k_pool, const void*
                                                  stream, dim3(1, 1, 1), p), "capped_attention (decode)");
     if (rc) return rc;
     if (splits > 1) {
-      rc = gb::check_pdl_launch(gb::launch_pdl(capped_attention_merge_kernel, dim3(Hkv, R), dim3(THREADS), 0, stream,
+      rc = gb::check_pdl_launch(gb::launch_pdl(capped_attention_merge_kernel, dim3(Hkv, R, min(max_q_len * g, ROWS_DECODE)), dim3(THREADS), 0, stream,
                                                dim3(1, 1, 1), p), "capped_attention (merge)");
       if (rc) return rc;
     }

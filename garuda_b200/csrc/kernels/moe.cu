@@ -22,9 +22,9 @@ route_topk_kernel(const HT* __restrict__ h, const WT* __restrict__ w, const floa
                   int K, int top, int mode, int32_t* __restrict__ ids, float* __restrict__ weights) {
   gb::pdl_launch_dependents();
   gb::pdl_wait();
-  extern __shared__ float sm[];        // z[E], then h[K]
-  float* z = sm;
-  float* h_s = sm + E;
+  extern __shared__ __align__(16) float sm[];        // h[K], then z[E]
+  float* h_s = sm;
+  float* z = sm + K;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   const int t = blockIdx.x;
   const HT* hr = h + (size_t)t * K;
@@ -33,7 +33,20 @@ route_topk_kernel(const HT* __restrict__ h, const WT* __restrict__ w, const floa
   for (int e = warp; e < E; e += warps) {
     const WT* wr = w + (size_t)e * K;
     float acc = 0.f;
-    for (int k = lane; k < K; k += 32) acc = fmaf(h_s[k], gb::to_float<WT>(wr[k]), acc);
+    if (sizeof(WT) == 2 && K % 8 == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0) {        // eight neighbouring weights in one load (rows start on 16 bytes)
+#pragma unroll 4
+      for (int k = lane * 8; k < K; k += 256) {
+        const uint4 v = *reinterpret_cast<const uint4*>(wr + k);
+        const uint32_t pairs[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          acc = fmaf(h_s[k + 2 * i], __uint_as_float(pairs[i] << 16), acc);
+          acc = fmaf(h_s[k + 2 * i + 1], __uint_as_float(pairs[i] & 0xffff0000u), acc);
+        }
+      }
+    } else {
+      for (int k = lane; k < K; k += 32) acc = fmaf(h_s[k], gb::to_float<WT>(wr[k]), acc);
+    }
     acc = gb::warp_sum(acc);
     if (lane == 0) z[e] = acc + (bias ? bias[e] : 0.f);
   }

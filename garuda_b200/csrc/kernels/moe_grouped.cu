@@ -234,12 +234,14 @@ struct TanhNorm {
 };
 
 // x[t][n] += alpha * sum_j weights[t][j] * y[pair_row[t * top + j]][n], j in the router's order; weights null: all one
+// grid (T, shares of the row)
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ y, const int32_t* __restrict__ pair_row, const float* __restrict__ weights,
                    float* __restrict__ x, int top, int N, float alpha, const TanhNorm norm) {
   const int t = blockIdx.x;
-  for (int n = threadIdx.x; n < N; n += blockDim.x) {
+  for (int n = blockIdx.y * blockDim.x + threadIdx.x; n < N; n += blockDim.x * gridDim.y) {
     float total = 0.f;
+#pragma unroll 4
     for (int j = 0; j < top; ++j) {
       const int row = pair_row[(size_t)t * top + j];
       if (row >= 0) total = fmaf(weights ? weights[(size_t)t * top + j] : 1.0f, y[(size_t)row * N + n], total);
@@ -250,6 +252,9 @@ moe_combine_kernel(const float* __restrict__ y, const int32_t* __restrict__ pair
   }
 }
 
+
+// A few tokens: a row over several blocks, so that more than a handful of SMs work.
+dim3 combine_grid(int T, int N) { return dim3(T, T >= 256 ? 1 : (N + 255) / 256); }
 
 template <int WM, int WN, int MI, int NP, int MODE, typename OT, typename... Args>
 int launch_grouped(dim3 grid, cudaStream_t stream, const char* what, Args... args) {
@@ -334,7 +339,7 @@ GB_EXPORT int gb_moe_grouped(const void* h, const void* w_gate_up, const void* w
     rc = launch_grouped<1, 4, 1, 1, PLAIN, float>(grid_n, stream, "moe_down_grouped", ac, F, zero, none, 1, wd, d_group, y, N,
                                                  zero, N, F, te, t0, tr, nt, 0, 0, 0.f, 0, no_scale);
   if (rc != GB_OK) return rc;
-  moe_combine_kernel<<<T, 256, 0, stream>>>(y, pair_row, out_weights, x, top, N, alpha,
+  moe_combine_kernel<<<combine_grid(T, N), 256, 0, stream>>>(y, pair_row, out_weights, x, top, N, alpha,
                                             TanhNorm{(__nv_bfloat16*)norm_out, norm_w, norm_b, norm_alpha});
   return gb::check_launch("moe_combine");
 }
@@ -437,7 +442,7 @@ GB_EXPORT int gb_moe_combine(const float* y, const int32_t* pair_row, const floa
                              int N, float alpha, void* norm_out, const float* norm_w, const float* norm_b, float norm_alpha,
                              cudaStream_t stream) {
   if (T <= 0) return GB_OK;
-  moe_combine_kernel<<<T, 256, 0, stream>>>(y, pair_row, weights, x, top, N, alpha,
+  moe_combine_kernel<<<combine_grid(T, N), 256, 0, stream>>>(y, pair_row, weights, x, top, N, alpha,
                                             TanhNorm{(__nv_bfloat16*)norm_out, norm_w, norm_b, norm_alpha});
   return gb::check_launch("moe_combine");
 }
