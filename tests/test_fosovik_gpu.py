@@ -534,7 +534,7 @@ def _random_config(rng):
             "embedding": {"scale": pick([1.0, 3.0, 12.0])}, "norm": {"eps": pick([1e-5, 1e-6])}, "layers": layers}
 
 
-@pytest.mark.parametrize("seed", [2, 5, 11, 17])
+@pytest.mark.parametrize("seed", [2, 11])
 def test_configurations_drawn_at_random(seed, tmp_path):
     from garuda_b200.weights import write_random_model
     from tests.plain import fosovik_plain as fp
