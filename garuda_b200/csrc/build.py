@@ -44,6 +44,9 @@ KERNEL_LIBS: Dict[str, List[str]] = {
     "garuda_seq": ["post_norm.cu", "mingru.cu", "conv_qkv.cu"],
     # a state space with one decay per head and token: built when a model first needs it
     "garuda_ssd": ["state_space.cu"],
+    # norms on both sides of a sublayer, a matrix memory, the plain differential attention: built when a model
+    # first needs them
+    "garuda_memory": ["residual_norm.cu", "matrix_memory.cu", "attention_diff.cu"],
 }
 HOST_SOURCES = ["cache_manager.cpp", "scheduler.cpp", "step_batch.cpp", "bindings.cpp"]
 
@@ -165,7 +168,16 @@ def ssd_lib_name(state_dim: int, head_dim: int) -> str:
     return f"garuda_ssdc_n{int(state_dim)}_p{int(head_dim)}"
 
 
+def diff_attention_lib_name(map_dim: int, value_dim: int) -> str:
+    """The tensor-core differential attention is compiled per (width of one map, value width), when a
+    model first needs it."""
+    return f"garuda_dattn_k{int(map_dim)}_v{int(value_dim)}"
+
+
 def _lib_recipe(name: str):
+    if name.startswith("garuda_dattn_k"):
+        kd, vd = name[len("garuda_dattn_k"):].split("_v")
+        return ["attention_diff_mma.cu"], [f"-DGB_MAP_DIM={int(kd)}", f"-DGB_VALUE_DIM={int(vd)}"]
     if name.startswith("garuda_ssdc_n"):
         n, p = name[len("garuda_ssdc_n"):].split("_p")
         return ["ssd_chunk_mma.cu"], [f"-DGB_STATE_DIM={int(n)}", f"-DGB_HEAD_DIM={int(p)}"]
@@ -283,7 +295,7 @@ def load_host_module():
 
 
 def build_all(head_dims=(16, 32, 48, 64, 128), latent_sizes=((64, 32), (512, 64)), capped_sizes=((64, 64), (32, 48)),
-              ssd_sizes=((64, 32), (128, 64))) -> None:
+              ssd_sizes=((64, 32), (128, 64)), diff_sizes=((32, 64), (64, 128))) -> None:
     """Everything, for a build check."""
     host_module_path()
     for name in KERNEL_LIBS:
@@ -296,3 +308,5 @@ def build_all(head_dims=(16, 32, 48, 64, 128), latent_sizes=((64, 32), (512, 64)
         kernel_lib_path(capped_attention_lib_name(kd, vd))
     for n, p in ssd_sizes:
         kernel_lib_path(ssd_lib_name(n, p))
+    for kd, vd in diff_sizes:
+        kernel_lib_path(diff_attention_lib_name(kd, vd))

@@ -244,7 +244,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __g
         __syncwarp();
       }
       if (!gave_up) {
-        process_tile<HD, SwizzledTile<HD, TK>, TK>(st, qf, SwizzledTile<HD, TK>{ks}, SwizzledTile<HD, TK>{vs}, key0, row_pos,
+        process_tile<HD, TK>(st, qf, SwizzledTile<HD, TK>{ks}, SwizzledTile<HD, TK>{vs}, key0, row_pos,
                                                    row_start, p.scale_log2, false);
         __syncwarp();             // every lane is done with the stage before it is filled again
         issue(t + DEPTH);

@@ -80,10 +80,11 @@ struct WarpState {
 // row_pos / row_start: last and first key each of the thread's two rows may read; full: every key
 // of the tile is inside every row's range (no mask needed). The running maximum st.m is kept
 // unscaled (a raw dot product); the merges scale it.
-// KEYS: keys in the tile (64, or 32 for the smaller tiles of the decode kernel that copies by TMA).
-template <int HD, typename Tile, int KEYS = KT>
-__device__ __forceinline__ void process_tile(WarpState<HD>& st, const uint32_t (&qf)[HD / 16][4],
-                                             const Tile ks, const Tile vs, int key0,
+// KEYS: keys in the tile (64, or fewer for the smaller tiles of the decode kernels). VD: the values' width, where it is
+// not the keys'.
+template <int HD, int KEYS = KT, int VD, typename KeyTile, typename ValueTile>
+__device__ __forceinline__ void process_tile(WarpState<VD>& st, const uint32_t (&qf)[HD / 16][4],
+                                             const KeyTile ks, const ValueTile vs, int key0,
                                              const int (&row_pos)[2], const int (&row_start)[2], float scale_log2,
                                              bool full) {
   const int lane = threadIdx.x & 31;
@@ -149,14 +150,14 @@ __device__ __forceinline__ void process_tile(WarpState<HD>& st, const uint32_t (
 #pragma unroll
   for (int i = 0; i < 2; ++i) st.l[i] = st.l[i] * corr[i] + l_add[i];
 #pragma unroll
-  for (int n = 0; n < HD / 8; ++n) {
+  for (int n = 0; n < VD / 8; ++n) {
     st.o[n][0] *= corr[0]; st.o[n][1] *= corr[0];
     st.o[n][2] *= corr[1]; st.o[n][3] *= corr[1];
   }
 #pragma unroll
   for (int kk = 0; kk < KEYS / 16; ++kk) {
 #pragma unroll
-    for (int n2 = 0; n2 < HD / 16; ++n2) {
+    for (int n2 = 0; n2 < VD / 16; ++n2) {
       uint32_t b[4];
       const int key = kk * 16 + (lane % 8) + ((lane / 8) % 2) * 8;
       ldmatrix_x4_trans(b, vs.chunk(key, n2 * 2 + (lane / 16)));

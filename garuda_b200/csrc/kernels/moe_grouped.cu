@@ -233,18 +233,22 @@ struct TanhNorm {
   float alpha;
 };
 
-// x[t][n] += alpha * sum_j weights[t][j] * y[pair_row[t * top + j]][n], j in the router's order; weights null: all one
+// x[t][n] += alpha * sum_j weights[t][j] * y[pair_row[t * top + j]][n], j in the router's order; weights null: all one.
+// A pair without a row (its id is beyond the experts): identity[t][n] in its place (null: nothing).
 // grid (T, shares of the row)
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ y, const int32_t* __restrict__ pair_row, const float* __restrict__ weights,
-                   float* __restrict__ x, int top, int N, float alpha, const TanhNorm norm) {
+                   float* __restrict__ x, int top, int N, float alpha, const TanhNorm norm,
+                   const __nv_bfloat16* __restrict__ identity) {
   const int t = blockIdx.x;
   for (int n = blockIdx.y * blockDim.x + threadIdx.x; n < N; n += blockDim.x * gridDim.y) {
     float total = 0.f;
 #pragma unroll 4
     for (int j = 0; j < top; ++j) {
       const int row = pair_row[(size_t)t * top + j];
-      if (row >= 0) total = fmaf(weights ? weights[(size_t)t * top + j] : 1.0f, y[(size_t)row * N + n], total);
+      const float wt = weights ? weights[(size_t)t * top + j] : 1.0f;
+      if (row >= 0) total = fmaf(wt, y[(size_t)row * N + n], total);
+      else if (identity != nullptr) total = fmaf(wt, __bfloat162float(identity[(size_t)t * N + n]), total);
     }
     const float v = fmaf(alpha, total, x[(size_t)t * N + n]);
     x[(size_t)t * N + n] = v;
@@ -286,8 +290,10 @@ GB_EXPORT long long gb_moe_grouped_index_words(long long R, int E) {
 GB_EXPORT int gb_moe_grouped(const void* h, const void* w_gate_up, const void* w_down, const int32_t* ids,
                              const float* weights, float* x, int T, int top, int E, int F, int K, int N, int kind,
                              float limit, float alpha, int layout, int scale_input, int32_t* index, void* act, float* y,
-                             void* norm_out, const float* norm_w, const float* norm_b, float norm_alpha, cudaStream_t stream) {
+                             void* norm_out, const float* norm_w, const float* norm_b, float norm_alpha, int identity,
+                             cudaStream_t stream) {
   if (T <= 0) return GB_OK;
+  if (identity && (K != N || scale_input)) return gb::fail(GB_BAD_ARGUMENT, "moe_grouped: an expert that returns its input of %d for outputs of %d", K, N);
   if (K % 8 || F % 8) return gb::fail(GB_UNSUPPORTED, "moe_grouped: widths %d and %d must be multiples of 8", K, F);
   if (E < 1 || (size_t)E * 2 * sizeof(int32_t) > 40 * 1024) return gb::fail(GB_UNSUPPORTED, "moe_grouped: %d experts", E);
   if (layout < 0 || layout > 2) return gb::fail(GB_BAD_ARGUMENT, "moe_grouped: layout %d", layout);
@@ -340,7 +346,7 @@ GB_EXPORT int gb_moe_grouped(const void* h, const void* w_gate_up, const void* w
                                                  zero, N, F, te, t0, tr, nt, 0, 0, 0.f, 0, no_scale);
   if (rc != GB_OK) return rc;
   moe_combine_kernel<<<combine_grid(T, N), 256, 0, stream>>>(y, pair_row, out_weights, x, top, N, alpha,
-                                            TanhNorm{(__nv_bfloat16*)norm_out, norm_w, norm_b, norm_alpha});
+                                            TanhNorm{(__nv_bfloat16*)norm_out, norm_w, norm_b, norm_alpha}, identity ? hh : nullptr);
   return gb::check_launch("moe_combine");
 }
 
@@ -438,12 +444,13 @@ GB_EXPORT int gb_moe_padded_prepare(const void* h, const int32_t* ids, int T, in
 
 // x[t] += alpha * sum_j weights[t][j] * y[pair_row[t * top + j]], j in the router's order; norm_out (or null): also
 // tanh(norm_alpha x) norm_w + norm_b of the new x, bfloat16 (likewise for gb_moe_grouped)
+// identity: [T, N] bfloat16 or null, the rows that pairs without an expert's row stand for.
 GB_EXPORT int gb_moe_combine(const float* y, const int32_t* pair_row, const float* weights, float* x, int T, int top,
                              int N, float alpha, void* norm_out, const float* norm_w, const float* norm_b, float norm_alpha,
-                             cudaStream_t stream) {
+                             const void* identity, cudaStream_t stream) {
   if (T <= 0) return GB_OK;
   moe_combine_kernel<<<combine_grid(T, N), 256, 0, stream>>>(y, pair_row, weights, x, top, N, alpha,
-                                            TanhNorm{(__nv_bfloat16*)norm_out, norm_w, norm_b, norm_alpha});
+                                            TanhNorm{(__nv_bfloat16*)norm_out, norm_w, norm_b, norm_alpha}, (const __nv_bfloat16*)identity);
   return gb::check_launch("moe_combine");
 }
 

@@ -17,6 +17,10 @@
 // which accumulators are again operands, and nothing of S is ever exchanged; the shares of y are added up in
 // shared memory. The next chunk is on its way (cp.async) while one is computed.
 //
+// A sum of many log decays loses the low bits of the differences that the products take, so L_i is kept as two floats.
+// A head may keep one more row of state whose input is the constant one (the normalizer of a matrix memory): a slice
+// of its own, of which one row counts.
+//
 // Compiled per (GB_STATE_DIM = channels of S, GB_HEAD_DIM = rows of S), multiples of 16.
 #include "attention_mma_core.cuh"
 #include "common.cuh"
@@ -56,7 +60,7 @@ struct Smem {
   };
   float grow[2][Q];                                // exp(L_i)
   float fade[2][Q];                                // exp(L_last - L_j) dt_j
-  float log_sum[2][Q];                             // L_i
+  float log_sum[2][Q], log_rest[2][Q];             // L_i, and what it lost in rounding
   float dt[2][Q];
 };
 
@@ -87,14 +91,15 @@ __device__ __forceinline__ int m_block(int warp, int k, int& ib, int& jb) {
   return 1;
 }
 
-// grid (H, P / PS, R). act [T, C]: x of all heads, B of all groups, C of all groups; step [T, 2 H]: dt, log of the decay.
+// grid (H, P / PS, one more for a unit row, R). act [T, C]: x of all heads, B of all groups, C of all groups; step [T, 2 H]: dt, log of the decay.
 __global__ void __launch_bounds__(THREADS, N <= 128 ? 2 : 1)
 ssd_chunk_kernel(const __nv_bfloat16* __restrict__ act, int C, const float* __restrict__ step, const float* __restrict__ skip,
                  const int32_t* __restrict__ cu_q, const int32_t* __restrict__ slots, float* __restrict__ state,
-                 long long state_stride, int H, int G, float* __restrict__ y) {
+                 long long state_stride, int H, int G, float* __restrict__ y, float* __restrict__ unit_state, float* __restrict__ unit_y) {
   extern __shared__ __align__(16) unsigned char raw[];
   Smem& sm = *reinterpret_cast<Smem*>(raw);
   gb::pdl_wait();
+  const bool unit = blockIdx.y == P / PS;
   const int h = blockIdx.x, p0 = blockIdx.y * PS, r = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tig = lane & 3;
   const int pr = warp % PR, kh = warp / PR;
@@ -112,7 +117,7 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ act, int C, const float* __re
       cp_async_16(&s.b[row][ch], src + off_b, ok);
       cp_async_16(&s.c[row][ch], src + off_c, ok);
     }
-    for (int i = threadIdx.x; i < Q * (PS / 8); i += THREADS) {
+    for (int i = threadIdx.x; i < (unit ? 0 : Q * (PS / 8)); i += THREADS) {
       const int row = i / (PS / 8), ch = (i % (PS / 8)) * 8;
       const bool ok = base + row < t1;
       cp_async_16(&s.x[row][ch], act + (size_t)(ok ? base + row : t0) * C + off_x + ch, ok);
@@ -132,29 +137,32 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ act, int C, const float* __re
     }
   };
   auto decays = [&](int st) {
-    float run = a[0] + a[1];
+    double run = (double)a[0] + a[1];
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
-      const float up = __shfl_up_sync(0xffffffffu, run, o);
+      const double up = __shfl_up_sync(0xffffffffu, run, o);
       if (lane >= o) run += up;
     }
-    const float last = __shfl_sync(0xffffffffu, run, 31);
-    float before = __shfl_up_sync(0xffffffffu, run, 1);
-    if (lane == 0) before = 0.f;
-    const float l[2] = {before + a[0], run};
+    const double last = __shfl_sync(0xffffffffu, run, 31);
+    double before = __shfl_up_sync(0xffffffffu, run, 1);
+    if (lane == 0) before = 0.0;
+    const double l[2] = {before + a[0], run};
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int i = 2 * lane + e;
-      sm.log_sum[st][i] = l[e];
+      sm.log_sum[st][i] = (float)l[e];
+      sm.log_rest[st][i] = (float)(l[e] - (float)l[e]);
       sm.dt[st][i] = d[e];
-      sm.grow[st][i] = expf(l[e]);
-      sm.fade[st][i] = expf(last - l[e]) * d[e];
+      sm.grow[st][i] = expf((float)l[e]);
+      sm.fade[st][i] = expf((float)(last - l[e])) * d[e];
     }
   };
 
   // the warp's piece of S^T: rows pr * 16 .., channel blocks kh, kh + KS, ...; two accumulator tiles of 8 channels each
   float S[MT][2][4];
-  float* S_g = slot >= 0 ? state + (size_t)slot * state_stride + ((size_t)h * P + p0 + pr * 16) * N : nullptr;
+  float* S_g = slot >= 0 ? (unit ? unit_state + (size_t)slot * state_stride + (size_t)h * N
+                                 : state + (size_t)slot * state_stride + ((size_t)h * P + p0 + pr * 16) * N) : nullptr;
+  const int S_rows = unit ? (pr == 0 ? 1 : 0) : 16;             // rows of the warp's piece that there are
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -162,9 +170,12 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ act, int C, const float* __re
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int n = (kh + m * KS) * 16 + half * 8 + 2 * tig + (e & 1), row = g + (e >> 1) * 8;
-        S[m][half][e] = (S_g != nullptr && kh + m * KS < NT) ? S_g[(size_t)row * N + n] : 0.f;
+        S[m][half][e] = (S_g != nullptr && row < S_rows && kh + m * KS < NT) ? S_g[(size_t)row * N + n] : 0.f;
       }
-  const float dskip = skip[h];
+  const float dskip = unit || skip == nullptr ? 0.f : skip[h];
+  if (unit)                       // its input, for every chunk (tokens beyond a request's last have step zero)
+    for (int i = threadIdx.x; i < 2 * Q * PS; i += THREADS)
+      sm.stage[i / (Q * PS)].x[i / PS % Q][i % PS] = __float2bfloat16_rn(i % PS == 0 ? 1.f : 0.f);
   const int chunks = (t1 - t0 + Q - 1) / Q;
   load(0, 0);
   if (warp == WARPS - 1) {
@@ -197,11 +208,11 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ act, int C, const float* __re
 #pragma unroll
         for (int up = 0; up < 2; ++up) {
           const int i = ib * 16 + g + up * 8, j = jb * 16 + half * 8 + 2 * tig;
-          const float li = sm.log_sum[st][i];
+          const float li = sm.log_sum[st][i], li_rest = sm.log_rest[st][i];
           float v[2];
 #pragma unroll
           for (int e = 0; e < 2; ++e)
-            v[e] = j + e <= i ? acc[half][up * 2 + e] * (expf(li - sm.log_sum[st][j + e]) * sm.dt[st][j + e]) : 0.f;
+            v[e] = j + e <= i ? acc[half][up * 2 + e] * (expf((li - sm.log_sum[st][j + e]) + (li_rest - sm.log_rest[st][j + e])) * sm.dt[st][j + e]) : 0.f;
           uint32_t parts[SPLIT];
           split_pair(v[0], v[1], parts);
 #pragma unroll
@@ -317,6 +328,10 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ act, int C, const float* __re
       __syncthreads();
     }
     const int n = min(Q, t1 - t0 - ck * Q);
+    if (unit) {
+      if (threadIdx.x < n) unit_y[(size_t)(t0 + ck * Q + threadIdx.x) * H + h] = sm.y[0][threadIdx.x][0] + sm.y[1][threadIdx.x][0];
+      continue;
+    }
     for (int i = threadIdx.x; i < n * PS; i += THREADS) {
       const int t = i / PS, p = i % PS;
       y[(size_t)(t0 + ck * Q + t) * H * P + off_x + p] = fmaf(dskip, __bfloat162float(s.x[t][p]), sm.y[0][t][p] + sm.y[1][t][p]);
@@ -331,7 +346,7 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ act, int C, const float* __re
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int n = (kh + m * KS) * 16 + half * 8 + 2 * tig + (e & 1), row = g + (e >> 1) * 8;
-          if (kh + m * KS < NT) S_g[(size_t)row * N + n] = S[m][half][e];
+          if (row < S_rows && kh + m * KS < NT) S_g[(size_t)row * N + n] = S[m][half][e];
         }
   }
 }
@@ -340,11 +355,14 @@ ssd_chunk_kernel(const __nv_bfloat16* __restrict__ act, int C, const float* __re
 
 GB_DEFINE_LAST_ERROR()
 
-// act [T, C] bfloat16 (16-byte aligned, C a multiple of 8), step [T, 2 H], y [T, H P]; state as for gb_ssd_recurrence.
+// act [T, C] bfloat16 (16-byte aligned, C a multiple of 8), step [T, 2 H], y [T, H P]; skip, state and the unit row as for
+// gb_ssd_recurrence.
 GB_EXPORT int gb_ssd_chunk(const void* act, const float* step, const float* skip, const int32_t* cu_q, const int32_t* slots,
-                           float* state, long long state_stride, int R, int H, int G, float* y, cudaStream_t stream) {
+                           float* state, long long state_stride, int R, int H, int G, float* y, float* unit_state, float* unit_y,
+                           cudaStream_t stream) {
   if (R <= 0) return GB_OK;
   if (H < 1 || G < 1 || H % G) return gb::fail(GB_BAD_ARGUMENT, "ssd_chunk: %d heads in %d groups", H, G);
+  if ((unit_state == nullptr) != (unit_y == nullptr)) return gb::fail(GB_BAD_ARGUMENT, "ssd_chunk: a unit row has a state and a read-out");
   if (R > 65535 || ((uintptr_t)act & 15)) return gb::fail(GB_UNSUPPORTED, "ssd_chunk: %d requests, rows at %p", R, act);
   static gb::OncePerDevice configured;
   if (configured.needed()) {
@@ -353,7 +371,8 @@ GB_EXPORT int gb_ssd_chunk(const void* act, const float* step, const float* skip
     configured.done();
   }
   const int C = H * P + 2 * G * N;
-  return gb::check_pdl_launch(gb::launch_after(ssd_chunk_kernel, dim3(H, P / PS, R), dim3(THREADS), sizeof(Smem), stream, dim3(1, 1, 1),
-                                               (const __nv_bfloat16*)act, C, step, skip, cu_q, slots, state, state_stride, H, G, y),
+  return gb::check_pdl_launch(gb::launch_after(ssd_chunk_kernel, dim3(H, P / PS + (unit_state != nullptr), R), dim3(THREADS), sizeof(Smem), stream,
+                                               dim3(1, 1, 1), (const __nv_bfloat16*)act, C, step, skip, cu_q, slots, state, state_stride, H, G, y,
+                                               unit_state, unit_y),
                               "ssd_chunk");
 }

@@ -139,34 +139,46 @@ ssd_prepare_kernel(const Conv cv, const float* __restrict__ d_rows, const float*
   }
 }
 
+// A head may keep one more row of state, driven by the constant input one in place of an x channel (the normalizer
+// of a matrix memory): `state` is its place for head 0 in slot 0 ([H, dim], the slots as far apart as those of S; null: no such row), `y`
+// [T, H] its read-out.
+struct UnitRow {
+  float* state;
+  float* y;
+};
+
 constexpr int REC_WARPS = 4, REC_ROWS = 4, REC_TOKENS = 8;        // rows of S per warp; tokens staged at a time
 
-// grid (H, R, ceil(vdim / 16)), 128 threads. A warp owns four rows of S; lane l holds the channels l, l + 32, ...
+// grid (H, R, ceil(vdim / 16), one more for a unit row), 128 threads. A warp owns four rows of S; lane l holds the channels l, l + 32, ...
 // of each. A token's B, C, x, dt and decay come through shared memory, eight tokens at a time.
 template <int PER, typename XT>
 __global__ void __launch_bounds__(REC_WARPS * 32)
 ssd_recurrence_kernel(const XT* __restrict__ act, int C, const float* __restrict__ step, const float* __restrict__ skip,
                       const int32_t* __restrict__ cu_q, const int32_t* __restrict__ slots, float* __restrict__ state,
-                      long long state_stride, int H, int G, int dim, int vdim, float* __restrict__ y) {
+                      long long state_stride, int H, int G, int dim, int vdim, float* __restrict__ y, const UnitRow unit) {
   gb::pdl_wait();
   constexpr int W = PER * 32;
   __shared__ float sb[REC_TOKENS][W], sc[REC_TOKENS][W], sx[REC_TOKENS][REC_WARPS * REC_ROWS], sdt[REC_TOKENS];
   __shared__ float s_keep[REC_TOKENS], s_change[REC_TOKENS];
-  const int h = blockIdx.x, r = blockIdx.y, p0 = blockIdx.z * REC_WARPS * REC_ROWS;
+  const bool is_unit = unit.state != nullptr && blockIdx.z == gridDim.z - 1;
+  const int h = blockIdx.x, r = blockIdx.y, p0 = is_unit ? 0 : blockIdx.z * REC_WARPS * REC_ROWS;
+  const int rows = is_unit ? 1 : vdim;             // of this block's state
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int slot = slots[r], t0 = cu_q[r], t1 = cu_q[r + 1];
   const int off_b = H * vdim + h / (H / G) * dim, off_c = off_b + G * dim;
   const int row0 = p0 + warp * REC_ROWS;
-  float* S_g = slot >= 0 ? state + (size_t)slot * state_stride + (size_t)h * vdim * dim : nullptr;
+  float* S_g = slot >= 0 ? (is_unit ? unit.state : state) + (size_t)slot * state_stride + (size_t)h * rows * dim : nullptr;
+  float* y_g = is_unit ? unit.y + h : y + (size_t)h * vdim;
+  const long long y_stride = is_unit ? H : (long long)H * vdim;
   float S[REC_ROWS][PER];
 #pragma unroll
   for (int i = 0; i < REC_ROWS; ++i)
 #pragma unroll
     for (int k = 0; k < PER; ++k) {
       const int c = lane + 32 * k;
-      S[i][k] = (S_g != nullptr && row0 + i < vdim && c < dim) ? S_g[(size_t)(row0 + i) * dim + c] : 0.f;
+      S[i][k] = (S_g != nullptr && row0 + i < rows && c < dim) ? S_g[(size_t)(row0 + i) * dim + c] : 0.f;
     }
-  const float dskip = skip[h];
+  const float dskip = is_unit || skip == nullptr ? 0.f : skip[h];
   for (int c0 = t0; c0 < t1; c0 += REC_TOKENS) {
     const int n = min(REC_TOKENS, t1 - c0);
     __syncthreads();
@@ -178,7 +190,8 @@ ssd_recurrence_kernel(const XT* __restrict__ act, int C, const float* __restrict
     }
     for (int i = threadIdx.x; i < n * REC_WARPS * REC_ROWS; i += blockDim.x) {
       const int tt = i / (REC_WARPS * REC_ROWS), p = i % (REC_WARPS * REC_ROWS);
-      sx[tt][p] = p0 + p < vdim ? gb::to_float<XT>(act[(size_t)(c0 + tt) * C + h * vdim + p0 + p]) : 0.f;
+      if (is_unit) sx[tt][p] = p == 0 ? 1.f : 0.f;
+      else sx[tt][p] = p0 + p < vdim ? gb::to_float<XT>(act[(size_t)(c0 + tt) * C + h * vdim + p0 + p]) : 0.f;
     }
     if (threadIdx.x < n) {
       const float* st = step + (size_t)(c0 + threadIdx.x) * 2 * H;
@@ -205,8 +218,8 @@ ssd_recurrence_kernel(const XT* __restrict__ act, int C, const float* __restrict
       float mine = acc[0];                 // lane i stores row i
 #pragma unroll
       for (int i = 1; i < REC_ROWS; ++i) mine = lane == i ? acc[i] : mine;
-      if (lane < REC_ROWS && row0 + lane < vdim)
-        y[(size_t)(c0 + tt) * H * vdim + h * vdim + row0 + lane] = fmaf(dskip, sx[tt][warp * REC_ROWS + lane], mine);
+      if (lane < REC_ROWS && row0 + lane < rows)
+        y_g[(c0 + tt) * y_stride + row0 + lane] = fmaf(dskip, sx[tt][warp * REC_ROWS + lane], mine);
     }
   }
   gb::pdl_launch_dependents();         // only now: the next kernel's blocks would wait beside these for the whole walk
@@ -216,7 +229,7 @@ ssd_recurrence_kernel(const XT* __restrict__ act, int C, const float* __restrict
 #pragma unroll
       for (int k = 0; k < PER; ++k) {
         const int c = lane + 32 * k;
-        if (row0 + i < vdim && c < dim) S_g[(size_t)(row0 + i) * dim + c] = S[i][k];
+        if (row0 + i < rows && c < dim) S_g[(size_t)(row0 + i) * dim + c] = S[i][k];
       }
   }
 }
@@ -409,20 +422,23 @@ GB_EXPORT int gb_ssd_prepare(const float* proj, long long P, int cx, int cd, con
   });
 }
 
-// Walks every request's tokens in order; y [T, H vdim].
+// Walks every request's tokens in order; y [T, H vdim]. skip null: no skip term. unit_state, unit_y: see UnitRow.
 GB_EXPORT int gb_ssd_recurrence(const void* act, int act_dtype, const float* step, const float* skip, const int32_t* cu_q,
                                 const int32_t* slots, float* state, long long state_stride, int R, int H, int G, int dim,
-                                int vdim, float* y, cudaStream_t stream) {
+                                int vdim, float* y, float* unit_state, float* unit_y, cudaStream_t stream) {
   if (R <= 0) return GB_OK;
   int rc = check_sizes("ssd_recurrence", H, G, dim, vdim, 1);
   if (rc != GB_OK) return rc;
+  if ((unit_state == nullptr) != (unit_y == nullptr)) return gb::fail(GB_BAD_ARGUMENT, "ssd_recurrence: a unit row has a state and a read-out");
+  if (R > 65535) return gb::fail(GB_UNSUPPORTED, "ssd_recurrence: %d requests", R);
+  const UnitRow unit = {unit_state, unit_y};
   const int rows = REC_WARPS * REC_ROWS, C = H * vdim + 2 * G * dim;
-  const dim3 grid(H, R, (vdim + rows - 1) / rows);
+  const dim3 grid(H, R, (vdim + rows - 1) / rows + (unit_state != nullptr));
   return GB_DISPATCH_DTYPE(act_dtype, XT, [&]() -> int {
     auto go = [&](auto per) -> int {
       return gb::check_pdl_launch(gb::launch_after(ssd_recurrence_kernel<decltype(per)::value, XT>, grid, dim3(REC_WARPS * 32), 0, stream,
                                                    dim3(1, 1, 1), (const XT*)act, C, step, skip, cu_q, slots, state, state_stride, H,
-                                                   G, dim, vdim, y),
+                                                   G, dim, vdim, y, unit),
                                   "ssd_recurrence");
     };
     if (dim <= 32) return go(std::integral_constant<int, 1>());

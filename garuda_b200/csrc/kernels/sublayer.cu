@@ -5,7 +5,8 @@
 //                        channel, rotation of the first channels) to q_out; keys (the same, one
 //                        weight for all heads) and values into their pages; the values may be the
 //                        keys' own columns as projected (before norm and rotation); queries may also be
-//                        multiplied by a number that grows with their position
+//                        multiplied by a number that grows with their position; a bias on every column;
+//                        neighbouring key heads side by side in one cached row
 //   gate_mul             x <- x * act(gate), act = sigmoid | silu, the gate's logits 32-bit
 //   unary_act            out = act(z), act = sigmoid | silu | relu^2 | tanh | exact gelu
 //   sublayer_merge       y = alpha * sum_b rms(y_b) * w_b   (or y = y_0)
@@ -28,7 +29,9 @@ qk_norm_rope_append_kernel(const float* __restrict__ src, int row_stride, int q_
                            const int32_t* __restrict__ positions, const int32_t* __restrict__ token_req,
                            const int32_t* __restrict__ block_table, int table_width, int Hq, int Hkv, int dim, int vdim,
                            const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
-                           const float* __restrict__ inv_freq, int interleaved, int page_size, float q_coef, int q_every) {
+                           const float* __restrict__ inv_freq, int interleaved, int rot_dims, float rot_factor, int page_size,
+                           float q_coef, int q_every, const float* __restrict__ bias, int maps) {
+  // maps: so many neighbouring key heads share a cached key row, [map 1 | map 2 ...], and one value
   __shared__ float sin_s[QK_MAX_DIM / 2], cos_s[QK_MAX_DIM / 2];
   gb::pdl_launch_dependents();
   gb::pdl_wait();
@@ -37,11 +40,19 @@ qk_norm_rope_append_kernel(const float* __restrict__ src, int row_stride, int q_
   const int half = dim >> 1;
   const bool rotate = inv_freq != nullptr;
   if (rotate)
-    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * inv_freq[i], &sin_s[i], &cos_s[i]);
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+      float sn = 0.f, cs = 1.f;                    // pairs beyond the rotated width stay as they are
+      if (i < rot_dims >> 1) {
+        sincosf((float)pos * inv_freq[i], &sn, &cs);
+        sn *= rot_factor, cs *= rot_factor;
+      }
+      sin_s[i] = sn, cos_s[i] = cs;
+    }
+  const int cached_heads = Hkv / maps;
   long long cache_row = -1;
   if (Hkv > 0) {
     const int page = block_table[(size_t)token_req[t] * table_width + pos / page_size];
-    if (page >= 0) cache_row = (long long)page * Hkv;       // no page behind this position: nothing is stored
+    if (page >= 0) cache_row = (long long)page * cached_heads;       // no page behind this position: nothing is stored
   }
   __syncthreads();
   const float* row = src + (size_t)t * row_stride;
@@ -56,20 +67,25 @@ qk_norm_rope_append_kernel(const float* __restrict__ src, int row_stride, int q_
     if (!is_q && cache_row < 0) continue;
     const float* s = row + (is_q ? q_col + head * dim : k_col + (head - Hq) * dim);
     const float* w = is_q ? (q_w ? q_w + (size_t)head * dim : nullptr) : k_w;
+    const float* bs = bias ? bias + (size_t)head * dim : nullptr;          // the keys' follow the queries'
     const bool normed = is_q ? q_w != nullptr : k_w != nullptr;
     float inv = 1.0f;
     if (normed) {
       float ss = 0.f;
-      for (int c = lane; c < dim; c += 32) ss = fmaf(s[c], s[c], ss);
+      for (int c = lane; c < dim; c += 32) {
+        const float v = s[c] + (bs ? bs[c] : 0.f);
+        ss = fmaf(v, v, ss);
+      }
       inv = 1.0f / sqrtf(gb::warp_sum(ss) / (float)dim + eps);
     }
     const float times = is_q ? growth : 1.0f;
     OT* dst = is_q ? q_out + ((size_t)t * Hq + head) * dim
-                   : k_pool + ((cache_row + (head - Hq)) * page_size + (pos % page_size)) * dim;
+                   : k_pool + ((cache_row + (head - Hq) / maps) * page_size + (pos % page_size)) * (maps * dim) + (head - Hq) % maps * dim;
     if (paired) {        // neighbours rotate together: one 8-byte load and one store for the two
       for (int i = lane; i < half; i += 32) {
         const float2 ab = *reinterpret_cast<const float2*>(s + 2 * i);
         float a = ab.x, b = ab.y;
+        if (bs) a += bs[2 * i], b += bs[2 * i + 1];
         if (normed) a = (a * inv) * w[2 * i], b = (b * inv) * w[2 * i + 1];
         if (rotate) {
           const float ra = a * cos_s[i] - b * sin_s[i], rb = b * cos_s[i] + a * sin_s[i];
@@ -79,10 +95,12 @@ qk_norm_rope_append_kernel(const float* __restrict__ src, int row_stride, int q_
       }
       continue;
     }
-    for (int i = lane; i < half; i += 32) {
+    const int turned = rotate && !interleaved ? rot_dims : dim & ~1;        // the channels that pairs cover
+    for (int i = lane; i < turned >> 1; i += 32) {
       const int ia = interleaved ? 2 * i : i;
-      const int ib = interleaved ? 2 * i + 1 : i + half;
+      const int ib = interleaved ? 2 * i + 1 : i + (turned >> 1);
       float a = s[ia], b = s[ib];
+      if (bs) a += bs[ia], b += bs[ib];
       if (normed) a = (a * inv) * w[ia], b = (b * inv) * w[ib];
       if (rotate) {
         const float ra = a * cos_s[i] - b * sin_s[i], rb = b * cos_s[i] + a * sin_s[i];
@@ -91,17 +109,18 @@ qk_norm_rope_append_kernel(const float* __restrict__ src, int row_stride, int q_
       dst[ia] = gb::from_float<OT>(a * times);
       dst[ib] = gb::from_float<OT>(b * times);
     }
-    if ((dim & 1) && lane == 0) {          // the last channel of an odd head has no partner (and no rotation)
-      float a = s[dim - 1];
-      if (normed) a = (a * inv) * w[dim - 1];
-      dst[dim - 1] = gb::from_float<OT>(a * times);
+    for (int c = turned + lane; c < dim; c += 32) {          // what no pair covers (the last channel of an odd head, too) passes
+      float a = s[c] + (bs ? bs[c] : 0.f);
+      if (normed) a = (a * inv) * w[c];
+      dst[c] = gb::from_float<OT>(a * times);
     }
   }
   if (cache_row >= 0) {
     const float* vs = row + v_col;
-    for (int e = threadIdx.x; e < Hkv * vdim; e += blockDim.x) {
+    const float* bs = bias ? bias + (size_t)(Hq + Hkv) * dim : nullptr;
+    for (int e = threadIdx.x; e < cached_heads * vdim; e += blockDim.x) {
       const int head = e / vdim, c = e % vdim;
-      v_pool[((cache_row + head) * page_size + (pos % page_size)) * vdim + c] = gb::from_float<OT>(vs[e]);
+      v_pool[((cache_row + head) * page_size + (pos % page_size)) * vdim + c] = gb::from_float<OT>(vs[e] + (bs ? bs[e] : 0.f));
     }
   }
 }
@@ -300,10 +319,12 @@ GB_EXPORT int gb_qk_norm_rope_append(const float* src, int row_stride, int q_col
                                      void* k_pool, void* v_pool, int out_dtype, const int32_t* positions,
                                      const int32_t* token_req, const int32_t* block_table, int table_width, int T, int Hq,
                                      int Hkv, int dim, int vdim, const float* q_w, const float* k_w, float eps,
-                                     const float* inv_freq, int interleaved, int page_size, float q_coef, int q_every,
-                                     cudaStream_t stream) {
+                                     const float* inv_freq, int interleaved, int rot_dims, float rot_factor, int page_size,
+                                     float q_coef, int q_every, const float* bias, int maps, cudaStream_t stream) {
   if (T <= 0) return GB_OK;
-  if (inv_freq != nullptr && (dim % 2 || dim > QK_MAX_DIM)) return gb::fail(GB_UNSUPPORTED, "qk_norm_rope_append: a rotated head of %d channels (even, at most %d)", dim, QK_MAX_DIM);
+  if (inv_freq != nullptr && (rot_dims % 2 || rot_dims < 2 || rot_dims > dim || dim > QK_MAX_DIM))
+    return gb::fail(GB_UNSUPPORTED, "qk_norm_rope_append: %d rotated channels of %d (even, heads of at most %d)", rot_dims, dim, QK_MAX_DIM);
+  if (maps < 1 || Hkv % maps) return gb::fail(GB_BAD_ARGUMENT, "qk_norm_rope_append: %d key heads, %d to a row", Hkv, maps);
   if (Hkv > 0 && (!k_pool || !v_pool || !block_table || page_size < 1))
     return gb::fail(GB_BAD_ARGUMENT, "qk_norm_rope_append: kv heads given without a cache to store them in");
   const int heads = Hq + Hkv;
@@ -312,7 +333,7 @@ GB_EXPORT int gb_qk_norm_rope_append(const float* src, int row_stride, int q_col
     return gb::check_pdl_launch(
         gb::launch_pdl(qk_norm_rope_append_kernel<OT>, dim3(T), dim3(block), 0, stream, dim3(1, 1, 1), src, row_stride, q_col,
                        k_col, v_col, (OT*)q_out, (OT*)k_pool, (OT*)v_pool, positions, token_req, block_table, table_width, Hq,
-                       Hkv, dim, vdim, q_w, k_w, eps, inv_freq, interleaved, page_size, q_coef, q_every),
+                       Hkv, dim, vdim, q_w, k_w, eps, inv_freq, interleaved, rot_dims, rot_factor, page_size, q_coef, q_every, bias, maps),
         "qk_norm_rope_append");
   });
 }

@@ -90,6 +90,7 @@ class CudaOps:
         self._state = None
         self._seq = None
         self._ssd = None
+        self._memory = None
         self._declare_core()
         # A word of pinned host memory that a kernel whose bounded wait ran out writes its code to (the
         # device reaches pinned host memory directly); ``failed_wait`` reads it without a copy.
@@ -214,11 +215,41 @@ class CudaOps:
             self._ssd = L
         return self._ssd
 
+    @property
+    def memory_lib(self):
+        """The library of the matrix-memory, differential-attention and two-sided-norm kernels, compiled and
+        loaded when a model first needs it."""
+        if self._memory is None:
+            L = load_kernel_lib("garuda_memory")
+            L.gb_last_error.restype = ctypes.c_char_p
+            for name, argtypes in self._MEMORY_SIGNATURES.items():
+                fn = getattr(L, name)
+                fn.argtypes = argtypes
+                fn.restype = c_int
+            self._memory = L
+        return self._memory
+
+    _MEMORY_SIGNATURES = {
+        "gb_residual_norm": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_float, c_void_p, c_int, c_longlong, c_int, c_int,
+                             c_void_p],
+        "gb_embedding_norm": [c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
+        "gb_memory_gates": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p,
+                            c_void_p, c_int, c_int, c_void_p],
+        "gb_memory_finish": [c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_float, c_float, c_void_p, c_int, c_int, c_int,
+                             c_int, c_void_p],
+        "gb_memory_decode": [c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_longlong,
+                             c_void_p, c_float, c_float, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_int,
+                             c_void_p],
+        "gb_diff_attention_simple": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                                     c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_float, c_float, c_float, c_void_p, c_longlong,
+                                     c_void_p],
+    }
+
     _SSD_SIGNATURES = {
         "gb_ssd_prepare": [c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p,
                            c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "gb_ssd_recurrence": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int,
-                              c_int, c_int, c_void_p, c_void_p],
+                              c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
         "gb_ssd_decode": [c_void_p, c_longlong, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_void_p,
                           c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
         "gb_ssd_finish": [c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int,
@@ -265,7 +296,7 @@ class CudaOps:
                              c_void_p],
         "gb_qk_norm_rope_append": [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                    c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float,
-                                   c_void_p, c_int, c_int, c_float, c_int, c_void_p],
+                                   c_void_p, c_int, c_int, c_float, c_int, c_float, c_int, c_void_p, c_int, c_void_p],
         "gb_gate_mul": [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
         "gb_unary_act": [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "gb_sublayer_merge": [c_void_p, c_void_p, c_int, c_float, c_float, c_void_p, c_int, c_void_p, c_void_p, c_float,
@@ -277,19 +308,19 @@ class CudaOps:
                                  c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
             "gb_head_gemm": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_int,
                              c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
-            "gb_route_topk": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                              c_void_p, c_void_p],
-            "gb_moe_gate_up": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+            "gb_route_topk": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
+                              c_int, c_void_p, c_void_p, c_void_p],
+            "gb_moe_gate_up": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                c_int, c_float, c_void_p, c_void_p],
-            "gb_moe_up": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                          c_void_p],
-            "gb_moe_down": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
-                            c_float, c_void_p],
-            "gb_moe_grouped": [c_void_p] * 6 + [c_int] * 7 + [c_float, c_float, c_int, c_int] + [c_void_p] * 6 + [c_float, c_void_p],
+            "gb_moe_up": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                          c_void_p, c_void_p],
+            "gb_moe_down": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                            c_float, c_void_p, c_void_p],
+            "gb_moe_grouped": [c_void_p] * 6 + [c_int] * 7 + [c_float, c_float, c_int, c_int] + [c_void_p] * 6 + [c_float, c_int, c_void_p],
             "gb_moe_padded_prepare": [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
                                       c_void_p, c_void_p],
             "gb_moe_combine": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p,
-                               c_float, c_void_p],
+                               c_float, c_void_p, c_void_p],
             "gb_grouped_gemm": [c_void_p, c_int, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_longlong,
                                 c_int, c_int, c_int, c_int, c_void_p],
             "gb_latent_query_prepare": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
@@ -326,10 +357,11 @@ class CudaOps:
                 _need(t.is_cuda, "kernel operands must live on the CUDA device")
 
     # ------------------------------------------------------------------ parts
-    def inv_freq(self, rotary) -> torch.Tensor:
+    def inv_freq(self, rotary, takes_factor: bool = False) -> torch.Tensor:
         """One frequency per pair of the head for a ``RotaryParams``: its own table if it has
-        one, else ``1 / theta^(2i/head_dim)`` in 32-bit (garuda/src/simd/mod.rs:199). Made once
-        per parameter set."""
+        one, else ``1 / theta^(2i/head_dim)`` in 32-bit (garuda/src/simd/mod.rs:199). Made once per
+        parameter set. ``takes_factor``: the caller's kernel knows a number on the cosines and sines."""
+        _need(takes_factor or rotary.factor == 1.0, "this kernel rotates without a number on the cosines and sines")
         if rotary not in self._inv_freq:
             from ..parts.rotary import rotary_frequencies
             self._inv_freq[rotary] = torch.from_numpy(rotary_frequencies(rotary)).to(self.device)
@@ -719,12 +751,18 @@ class CudaOps:
     # ------------------------------------------------------------------ routed experts
     ROUTER_SCORES = {"softmax_chosen": 0, "sigmoid": 1, "softmax_all": 2}
 
-    def route_topk(self, h, w_router, bias, top, ids, weights, score: str = "softmax_chosen"):
+    def route_topk(self, h, w_router, bias, top, ids, weights, score: str = "softmax_chosen", correction=None, groups=None):
         """Router logits ``h @ w_router^T + bias`` in 32-bit; ``ids[T, top]`` the experts with the
         largest logits (descending), ``weights[T, top]`` the softmax over those logits only, or
         (``score`` "sigmoid") each chosen expert's ``sigmoid(logit)``, not renormalized, or
-        (``"softmax_all"``) its share of the softmax over all experts' logits, not renormalized."""
-        self._on_device(h, w_router, bias, ids, weights)
+        (``"softmax_all"``) its share of the softmax over all experts' logits, not renormalized.
+        ``correction`` (32-bit ``[E]``, with the latter two scores): the choice is by score + correction, the
+        weights are the scores without it. ``groups = (count, keep)``: only experts of the ``keep`` best of ``count``
+        equal groups of neighbours can be chosen, a group's score being its best expert's."""
+        self._on_device(h, w_router, bias, ids, weights, correction)
+        _need(correction is None or (correction.dtype == torch.float32 and correction.is_contiguous()
+                                     and correction.numel() == w_router.shape[0]), "route_topk: a float32 correction [E]")
+        count, keep = groups if groups is not None else (0, 0)
         T, K = h.shape
         E = w_router.shape[0]
         _need(h.is_contiguous() and w_router.is_contiguous() and w_router.shape[1] == K, "route_topk: shapes")
@@ -733,7 +771,8 @@ class CudaOps:
         _need(bias is None or (bias.dtype == torch.float32 and bias.numel() == E), "route_topk: a float32 bias")
         self._check(self.mixers, self.mixers.gb_route_topk(
             h.data_ptr(), _tag(h, "router input"), w_router.data_ptr(), _ptr(bias), _tag(w_router, "router"),
-            T, E, K, int(top), self.ROUTER_SCORES[score], ids.data_ptr(), weights.data_ptr(), self._stream()), "route_topk")
+            T, E, K, int(top), self.ROUTER_SCORES[score], _ptr(correction), int(count), int(keep), ids.data_ptr(), weights.data_ptr(),
+            self._stream()), "route_topk")
 
     def moe_gate_up(self, h, w_gate_up, ids, act, kind: str, limit: float, in_scale=None):
         """``act[T, top, F]``: every token's gate/up products against its chosen experts'
@@ -747,20 +786,22 @@ class CudaOps:
               and w_gate_up.shape[2] == K and act.shape == (T, top, F2 // 2), "moe_gate_up: shapes")
         self._check(self.mixers, self.mixers.gb_moe_gate_up(
             h.data_ptr(), _tag(h, "h"), w_gate_up.data_ptr(), _tag(w_gate_up, "w"), ids.data_ptr(), act.data_ptr(),
-            _tag(act, "act"), T, top, F2 // 2, K, self.GATE_ACTS[kind], float(limit), _ptr(in_scale), self._stream()),
+            _tag(act, "act"), T, top, E, F2 // 2, K, self.GATE_ACTS[kind], float(limit), _ptr(in_scale), self._stream()),
             "moe_gate_up")
 
-    def moe_down(self, act, w_down, ids, weights, x, alpha: float = 1.0):
+    def moe_down(self, act, w_down, ids, weights, x, alpha: float = 1.0, identity=None):
         """``x[t] += alpha * sum_j weights[t, j] * (act[t, j] @ w_down[ids[t, j]]^T)``; ``weights``
-        None: all one."""
+        None: all one. ``identity`` (``[T, N]``, ``act``'s dtype): what an id beyond the experts stands for (None: nothing)."""
         self._on_device(act, w_down, ids, weights, x)
         T, top, F = act.shape
         E, N, _ = w_down.shape
         _need(act.is_contiguous() and w_down.is_contiguous() and w_down.shape[2] == F and x.shape == (T, N)
               and x.dtype == torch.float32 and x.is_contiguous(), "moe_down: shapes")
+        self._on_device(identity)
+        _need(identity is None or (identity.dtype == act.dtype and identity.is_contiguous() and identity.shape == x.shape), "moe_down: identity")
         self._check(self.mixers, self.mixers.gb_moe_down(
             act.data_ptr(), _tag(act, "act"), w_down.data_ptr(), _tag(w_down, "w"), ids.data_ptr(),
-            _ptr(weights), x.data_ptr(), T, top, F, N, float(alpha), self._stream()), "moe_down")
+            _ptr(weights), x.data_ptr(), T, top, E, F, N, float(alpha), _ptr(identity), self._stream()), "moe_down")
 
     def moe_up(self, h, w_up, ids, act, kind: str, in_scale=None):
         """``act[T, top, F]``: as ``moe_gate_up`` for experts without a gate, ``w_up [E, F, K]``, an activation
@@ -793,7 +834,8 @@ class CudaOps:
     GROUPED_TC_PAIRS = 1024
 
     def routed_feed_forward(self, ctx, h, w_gate_up, w_down, ids, weights, x, kind: str, limit: float,
-                            alpha: float = 1.0, scale_input: bool = False, gated: bool = True, then=None):
+                            alpha: float = 1.0, scale_input: bool = False, gated: bool = True, then=None,
+                            identity: bool = False):
         """``x[t] += alpha * sum_j weights[t, j] * expert_{ids[t, j]}(h[t])`` with the experts'
         weights stacked: ``w_gate_up`` from ``pack_expert_gate_up``, ``w_down [E, N, F]``. Without ``gated``:
         ``w_gate_up`` is ``[E, F, K]``, the up rows alone, and ``kind`` an activation of one value.
@@ -801,14 +843,16 @@ class CudaOps:
         (32-bit vectors) into ``out`` (bfloat16 ``[T, N]``), where the tensor-core kernels take the sizes; returns
         whether it did.
         ``scale_input``: the weight multiplies what goes into the expert instead,
-        ``sum_j expert(weights[t, j] * h[t])``."""
+        ``sum_j expert(weights[t, j] * h[t])``. An id beyond the ``E`` experts stands for no expert: its term is
+        ``weights[t, j] * h[t]`` with ``identity``, else nothing."""
+        _need(not identity or (h.shape[1] == w_down.shape[1] and not scale_input), "routed_feed_forward: an expert that returns its input")
         T, top = ids.shape
         E, N, F = w_down.shape
         K = h.shape[1]
         packed = getattr(w_gate_up, "gb_group", 0) == 64
         grouped = packed if gated else (self.tc is not None and h.dtype == torch.bfloat16 and K % 8 == 0 and F % 8 == 0 and E <= 4096)
         if grouped and T * top >= self.GROUPED_TC_PAIRS and self._routed_tcgen05(ctx, h, w_gate_up, w_down, ids, weights,
-                                                                                x, kind, limit, alpha, scale_input, gated, then):
+                                                                                x, kind, limit, alpha, scale_input, gated, then, identity):
             return then is not None
         norm = self._then_norm(then, T, N)
         if grouped:
@@ -828,14 +872,14 @@ class CudaOps:
                 h.data_ptr(), w_gate_up.data_ptr(), w_down.data_ptr(), ids.data_ptr(), weights.data_ptr(), x.data_ptr(),
                 T, top, E, F, K, N, self.GATE_ACTS[kind] if gated else self.UNARY_ACTS[kind], float(limit), float(alpha),
                 1 if gated else 2, int(scale_input), index.data_ptr(),
-                act.data_ptr(), y.data_ptr(), *norm, self._stream()), "moe_grouped", 4)
+                act.data_ptr(), y.data_ptr(), *norm, int(identity), self._stream()), "moe_grouped", 4)
             return then is not None
         act = ctx.ws.get("expert_act", (T, top, F), h.dtype)
         if gated:
             self.moe_gate_up(h, w_gate_up, ids, act, kind, limit, weights if scale_input else None)
         else:
             self.moe_up(h, w_gate_up, ids, act, kind, weights if scale_input else None)
-        self.moe_down(act, w_down, ids, None if scale_input else weights, x, alpha)
+        self.moe_down(act, w_down, ids, None if scale_input else weights, x, alpha, h if identity else None)
         return False
 
     def _then_norm(self, then, rows, width):
@@ -848,7 +892,7 @@ class CudaOps:
         return (out.data_ptr(), w.data_ptr(), b.data_ptr(), float(alpha))
 
     def _routed_tcgen05(self, ctx, h, w_gate_up, w_down, ids, weights, x, kind, limit, alpha, scale_input=False,
-                        gated=True, then=None) -> bool:
+                        gated=True, then=None, identity=False) -> bool:
         """Many pairs: sorted by expert into blocks of 128 rows (padding rows zero), then the two
         products on the tcgen05 many-token kernel with each block's expert read from a list."""
         T, top = ids.shape
@@ -883,7 +927,8 @@ class CudaOps:
             tc.grouped(a, w_gate_up, act, F, E, block_gu, 0, gate_act=tc.STORE_ACTS[kind])
         tc.grouped(act, w_down, y, N, E, block_dn, 0)
         self._check(L, L.gb_moe_combine(y.data_ptr(), index.data_ptr(), None if scale_input else weights.data_ptr(), x.data_ptr(), T, top, N,
-                                        float(alpha), *self._then_norm(then, T, N), self._stream()), "moe_combine")
+                                        float(alpha), *self._then_norm(then, T, N), h.data_ptr() if identity else None, self._stream()),
+                    "moe_combine")
         return True
 
     # ------------------------------------------------------------------ attention over a cached latent
@@ -1140,7 +1185,7 @@ class CudaOps:
 
     # ------------------------------------------------------------------ normed queries and keys; sublayers normed behind
     def qk_norm_rope_append(self, src, cols, q_out, k_pool, v_pool, positions, token_req, block_table, heads, kv_heads,
-                            dim, vdim, q_weight, k_weight, eps, rotary, page_size, query_growth=None):
+                            dim, vdim, q_weight, k_weight, eps, rotary, page_size, query_growth=None, bias=None, maps: int = 1):
         """From a projected 32-bit row ``src [T, P]`` with ``cols = (q, k, v)`` the first columns of
         queries (``heads dim``), keys (``kv_heads dim``) and values (``kv_heads vdim``; the keys' own
         columns where the values are the keys as projected): queries and keys are divided by their root
@@ -1148,33 +1193,41 @@ class CudaOps:
         then rotated (``rotary``: a ``RotaryParams`` over ``dim``, or None); queries go to ``q_out
         [T, heads, dim]``, keys and the untouched values into their pages. ``query_growth = (coef, every)``: the
         query at position ``p`` is multiplied by ``1 + coef ln(floor((p + 1) / every) + 1)``. ``kv_heads`` 0: queries
-        only, the pools are not touched."""
-        self._on_device(src, q_out, k_pool, v_pool, positions, token_req, block_table, q_weight, k_weight)
+        only, the pools are not touched. A ``rotary`` narrower than ``dim`` turns the first channels; its ``factor``
+        multiplies cosines and sines. ``bias`` (32-bit, over the columns q | k | v): added first. ``maps`` n: n
+        neighbouring key heads lie side by side in one cached row, ``k_pool [pages, kv_heads / n, page_size, n dim]``,
+        beside one value head."""
+        self._on_device(bias, src, q_out, k_pool, v_pool, positions, token_req, block_table, q_weight, k_weight)
         T = src.shape[0]
         cq, ck, cv = (int(c) for c in cols)
+        cached = kv_heads // maps
+        _need(maps >= 1 and cached * maps == kv_heads, "qk_norm_rope_append: whole rows of key heads")
+        _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous()
+                               and bias.numel() == (heads + kv_heads) * dim + cached * vdim), "qk_norm_rope_append: a float32 bias over q | k | v")
         _need(src.dtype == torch.float32 and src.stride(1) == 1, "qk_norm_rope_append: a float32 row")
-        _need(max(cq + heads * dim, ck + kv_heads * dim, cv + kv_heads * vdim) <= src.shape[1], "qk_norm_rope_append: columns")
+        _need(max(cq + heads * dim, ck + kv_heads * dim, cv + cached * vdim) <= src.shape[1], "qk_norm_rope_append: columns")
         _need(q_out.is_contiguous() and tuple(q_out.shape) == (T, heads, dim), "qk_norm_rope_append: q_out shape")
         _need(kv_heads == 0 or (k_pool.dtype == q_out.dtype == v_pool.dtype and k_pool.is_contiguous() and v_pool.is_contiguous()
-              and tuple(k_pool.shape[1:]) == (kv_heads, page_size, dim)
-              and tuple(v_pool.shape[1:]) == (kv_heads, page_size, vdim)), "qk_norm_rope_append: pool shapes")
+              and tuple(k_pool.shape[1:]) == (cached, page_size, maps * dim)
+              and tuple(v_pool.shape[1:]) == (cached, page_size, vdim)), "qk_norm_rope_append: pool shapes")
         _need(block_table.dtype == torch.int32 and block_table.is_contiguous() and positions.dtype == torch.int32
               and token_req.dtype == torch.int32, "qk_norm_rope_append: int32 indices")
         _need(q_weight is None or (q_weight.dtype == torch.float32 and q_weight.is_contiguous()
                                    and q_weight.numel() == heads * dim), "qk_norm_rope_append: q_weight float32 [heads, dim]")
         _need(k_weight is None or (k_weight.dtype == torch.float32 and k_weight.is_contiguous()
                                    and k_weight.numel() == dim), "qk_norm_rope_append: k_weight float32 [dim]")
-        inv, inter = None, 0
+        inv, inter, turned, factor = None, 0, 0, 1.0
         if rotary is not None:
-            _need(rotary.head_dim == dim, "qk_norm_rope_append: rotary is for another head width")
-            inv, inter = self.inv_freq(rotary), int(rotary.interleaved)
+            _need(rotary.head_dim <= dim, "qk_norm_rope_append: rotary is for a wider head")
+            inv, inter = self.inv_freq(rotary, takes_factor=True), int(rotary.interleaved)
+            turned, factor = rotary.head_dim, float(rotary.factor)
         coef, every = query_growth if query_growth is not None else (0.0, 0)
         L = self.state_lib
         self._check(L, L.gb_qk_norm_rope_append(
             src.data_ptr(), src.stride(0), cq, ck, cv, q_out.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(),
             _tag(q_out, "q_out"), positions.data_ptr(), token_req.data_ptr(), block_table.data_ptr(), block_table.shape[1],
-            T, heads, kv_heads, dim, vdim, _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(inv), inter, page_size,
-            float(coef), int(every), self._stream()), "qk_norm_rope_append")
+            T, heads, kv_heads, dim, vdim, _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(inv), inter, turned, factor,
+            page_size, float(coef), int(every), _ptr(bias), int(maps), self._stream()), "qk_norm_rope_append")
 
     UNARY_ACTS = {"sigmoid": 0, "silu": 1, "relu2": 2, "tanh": 3, "gelu": 4}
 
@@ -1383,10 +1436,117 @@ class CudaOps:
                     act, step, skip, b.cu_q, b.slots, state, b.num_requests, H, G, dim, vdim, y)):
                 self._check(L, L.gb_ssd_recurrence(
                     act.data_ptr(), tag, step.data_ptr(), skip.data_ptr(), b.cu_q.data_ptr(), b.slots.data_ptr(), state.data_ptr(),
-                    stride, b.num_requests, H, G, dim, vdim, y.data_ptr(), self._stream()), "ssd_recurrence")
+                    stride, b.num_requests, H, G, dim, vdim, y.data_ptr(), None, None, self._stream()), "ssd_recurrence")
         self._check(L, L.gb_ssd_finish(
             y.data_ptr(), proj.data_ptr(), P, cz, cx, norm_w.data_ptr(), float(eps), out.data_ptr(), tag, T, int(norm_groups), inner,
             kept, stride, b.cu_q.data_ptr(), b.slots.data_ptr(), b.num_requests, C, taps, self._stream()), "ssd_finish")
+
+    # ------------------------------------------------------------------ a matrix memory with exponential gates
+    def matrix_memory(self, ctx, act, gates, bias_i, bias_f, cap, norm_w, scale, eps, state, heads, dim, vdim, out):
+        """The recurrent part of a matrix-memory mixer for one step. ``act [T, >= H vdim + 2 H dim]``: the projected v |
+        k | q of all heads, in ``out``'s dtype, or (steps of one token per request) as 32-bit rows, which are
+        rounded to it; ``gates [T, >= H vdim + 2 H]`` (32-bit): the output gate's, then the input and the forget
+        gate's logits. Per head: ``i = cap tanh((z_i + bias_i) / cap)``, ``f = log sigmoid(cap tanh((z_f + bias_f) /
+        cap))``, ``m' = max(f + m, i)``, ``S <- exp(f + m - m') S + exp(i - m') v k^T``, ``n`` likewise with ``k``, ``o = scale S q /
+        (max(|scale n . q|, exp(-m')) + 1e-6)``, ``out = o / rms(o) * norm_w * sigmoid(gate)``. ``state [slots, >= H vdim dim +
+        H dim + H]`` (32-bit: ``S [H, vdim, dim]``, ``n``, ``m``) is advanced for the batch's requests."""
+        b = ctx.batch
+        self._on_device(act, gates, bias_i, bias_f, norm_w, state, out)
+        T, H = out.shape[0], int(heads)
+        HP, HN = H * vdim, H * dim
+        _need(act.stride(1) == 1 and act.shape[0] == T and act.shape[1] >= HP + 2 * HN, "matrix_memory: rows of v, k, q")
+        _need(gates.dtype == torch.float32 and gates.stride(1) == 1 and gates.shape[0] == T and gates.shape[1] >= HP + 2 * H,
+              "matrix_memory: float32 rows of gates")
+        _need(all(v.dtype == torch.float32 and v.is_contiguous() for v in (bias_i, bias_f, norm_w)) and bias_i.numel() == bias_f.numel() == H
+              and norm_w.numel() == HP, "matrix_memory: float32 vectors")
+        _need(state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] >= HP * dim + HN + H, "matrix_memory: state")
+        _need(out.is_contiguous() and tuple(out.shape) == (T, HP), "matrix_memory: out")
+        L, stride, tag = self.memory_lib, state.shape[1], _tag(out, "matrix_memory out")
+        z_i = gates.data_ptr() + 4 * HP
+        z_f = z_i + 4 * H
+        if b.max_q_len == 1:
+            _need(act.dtype == torch.float32, "matrix_memory: float32 rows where every request brings one token")
+            self._check(L, L.gb_memory_decode(
+                act.data_ptr(), act.stride(0), z_i, z_f, gates.stride(0), bias_i.data_ptr(), bias_f.data_ptr(), float(cap), gates.data_ptr(),
+                gates.stride(0), norm_w.data_ptr(), float(scale), float(eps), b.slots.data_ptr(), state.data_ptr(), stride, T, H, dim,
+                vdim, out.data_ptr(), tag, self._stream()), "memory_decode")
+            return
+        _need(act.dtype == out.dtype and act.is_contiguous() and act.shape[1] == HP + 2 * HN, "matrix_memory: contiguous rows in out's dtype")
+        n_state = state.data_ptr() + 4 * HP * dim
+        step, floor = ctx.ws.get("memory_step", (T, 2 * H), torch.float32), ctx.ws.get("memory_floor", (T, H), torch.float32)
+        y, den = ctx.ws.get("memory_y", (T, HP), torch.float32), ctx.ws.get("memory_den", (T, H), torch.float32)
+        self._check(L, L.gb_memory_gates(
+            z_i, z_f, gates.stride(0), bias_i.data_ptr(), bias_f.data_ptr(), float(cap), b.cu_q.data_ptr(), b.slots.data_ptr(),
+            n_state + 4 * HN, stride, step.data_ptr(), floor.data_ptr(), b.num_requests, H, self._stream()), "memory_gates")
+        # the memory is a state space whose decays and steps are now known, the normalizer its row of constant input
+        if not (b.max_q_len >= self.SSD_CHUNK_TOKENS and self.tc is not None and self.tc.ssd_chunk(
+                act, step, None, b.cu_q, b.slots, state, b.num_requests, H, H, dim, vdim, y, n_state, den)):
+            S = self.ssd_lib
+            self._check(S, S.gb_ssd_recurrence(
+                act.data_ptr(), tag, step.data_ptr(), None, b.cu_q.data_ptr(), b.slots.data_ptr(), state.data_ptr(), stride,
+                b.num_requests, H, H, dim, vdim, y.data_ptr(), n_state, den.data_ptr(), self._stream()), "ssd_recurrence")
+        self._check(L, L.gb_memory_finish(
+            y.data_ptr(), den.data_ptr(), floor.data_ptr(), gates.data_ptr(), gates.stride(0), norm_w.data_ptr(), float(scale), float(eps),
+            out.data_ptr(), tag, T, H, vdim, self._stream()), "memory_finish")
+
+    # ------------------------------------------------------------------ norms on both sides of a sublayer
+    def residual_norm(self, x, y=None, weight=None, eps: float = 0.0, row=None, then_weight=None, then_eps: float = 0.0, out=None):
+        """``x += rms(y) * weight`` (``weight`` None: ``x += y``) and ``x += row`` on the 32-bit residual ``x [T, d]``, ``y`` 32-bit
+        ``[T, d]`` or None, ``row [d]`` or None; then ``out = rms(x) * then_weight`` (``then_weight`` None: ``out = x``) in
+        ``out``'s dtype (a column range of a wider row will do). Vectors are 32-bit. One pass."""
+        self._on_device(x, y, weight, row, then_weight, out)
+        _need(x.dtype == torch.float32 and x.is_contiguous() and x.dim() == 2, "residual_norm: x must be float32 [T, d]")
+        T, d = x.shape
+        _need(y is None or (y.dtype == torch.float32 and y.is_contiguous() and tuple(y.shape) == (T, d)), "residual_norm: y must be float32 of x's shape")
+        _need(all(v is None or (v.dtype == torch.float32 and v.is_contiguous() and v.numel() == d) for v in (weight, row, then_weight)),
+              "residual_norm: float32 vectors [d]")
+        _need(out is None or (tuple(out.shape) == (T, d) and out.stride(1) == 1), "residual_norm: out [T, d]")
+        L = self.memory_lib
+        self._check(L, L.gb_residual_norm(
+            x.data_ptr(), _ptr(y), _ptr(weight), float(eps), _ptr(row), _ptr(then_weight), float(then_eps), _ptr(out),
+            _tag(out, "residual_norm out") if out is not None else GB_F32, out.stride(0) if out is not None else d, T, d, self._stream()),
+            "residual_norm")
+
+    def embedding_norm(self, table, ids, weight, eps, x, pair=None):
+        """``x[t] = rms(table[ids[t]]) * weight`` in 32-bit; ``pair [T, 2 d]``: also ``[x | x]`` in its dtype."""
+        self._on_device(table, ids, weight, x, pair)
+        T, d = x.shape
+        _need(x.dtype == torch.float32 and x.is_contiguous() and ids.dtype == torch.int32 and ids.shape[0] == T, "embedding_norm: x, ids")
+        _need(table.is_contiguous() and table.shape[1] == d and weight.dtype == torch.float32 and weight.is_contiguous()
+              and weight.numel() == d, "embedding_norm: table, weight")
+        _need(pair is None or (pair.is_contiguous() and tuple(pair.shape) == (T, 2 * d)), "embedding_norm: pair")
+        L = self.memory_lib
+        self._check(L, L.gb_embedding_norm(
+            table.data_ptr(), _tag(table, "embedding table"), ids.data_ptr(), weight.data_ptr(), float(eps), x.data_ptr(), _ptr(pair),
+            _tag(pair, "pair") if pair is not None else GB_F32, T, d, table.shape[0], self._stream()), "embedding_norm")
+
+    # ------------------------------------------------------------------ two softmax maps over the same values
+    def differential_attention(self, ctx, q, k_pool, v_pool, block_table, out, scale, window, page_size, lam, out_scale, eps, gate=None):
+        """``q [T, H, 2 dim]`` and ``k_pool [pages, G, page_size, 2 dim]`` hold a head's two maps side by side, ``v_pool
+        [pages, G, page_size, vd]``. Per head: ``o = sum_j (p1_j - lam p2_j) v_j`` with each map's softmax over the keys
+        ``0 <= i - j < window`` (0: every ``j <= i``) of its scores times ``scale``; ``out = o / sqrt(mean(o^2) + eps) *
+        out_scale * sigmoid(gate)``, ``out [T, H vd]``, ``gate`` 32-bit logits ``[T, H]`` (a column range will do) or None."""
+        b = ctx.batch
+        self._on_device(q, k_pool, v_pool, block_table, out, gate)
+        T, H, D2 = q.shape
+        G, vd = k_pool.shape[1], v_pool.shape[3]
+        _need(D2 % 2 == 0 and q.is_contiguous() and out.is_contiguous() and tuple(out.shape) == (T, H * vd) and H % G == 0,
+              "differential_attention: q/out shape")
+        _need(q.dtype == k_pool.dtype == v_pool.dtype == out.dtype, "differential_attention: one dtype for q, cache and out")
+        _need(tuple(k_pool.shape[1:]) == (G, page_size, D2) and tuple(v_pool.shape[:3]) == tuple(k_pool.shape[:3])
+              and k_pool.is_contiguous() and v_pool.is_contiguous(), "differential_attention: pool shape")
+        _need(block_table.dtype == torch.int32 and block_table.is_contiguous(), "differential_attention: block table")
+        _need(gate is None or (gate.dtype == torch.float32 and tuple(gate.shape) == (T, H) and gate.stride(1) == 1),
+              "differential_attention: float32 gate logits [T, H]")
+        if self.tc is not None and q.dtype == torch.bfloat16 and self.tc.differential_attention(
+                q, k_pool, v_pool, block_table, b, out, scale, window, page_size, lam, out_scale, eps, gate, ctx.ws):
+            return
+        L = self.memory_lib
+        self._check(L, L.gb_diff_attention_simple(
+            q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), _tag(q, "differential_attention q"), block_table.data_ptr(),
+            block_table.shape[1], b.cu_q.data_ptr(), b.kv_lens.data_ptr(), b.token_req.data_ptr(), out.data_ptr(), T, H, G, D2 // 2, vd,
+            float(scale), int(window), int(page_size), float(lam), float(out_scale), float(eps), _ptr(gate),
+            gate.stride(0) if gate is not None else 0, self._stream()), "diff_attention")
 
     # ------------------------------------------------------------------ a short convolution in front of attention
     def conv_qkv_append(self, ctx, proj, bias, conv_w, taps, state, q_out, k_pool, v_pool, block_table, heads, kv_heads,

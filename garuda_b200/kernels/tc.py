@@ -12,7 +12,7 @@ from ctypes import c_void_p, c_int, c_float
 import torch
 
 from ..csrc.build import (load_kernel_lib, attention_lib_name, latent_attention_lib_name, capped_attention_lib_name,
-                          ssd_lib_name)
+                          ssd_lib_name, diff_attention_lib_name)
 
 _WAIT_NAMES = {1: "an operand tile never arrived (TMA)", 2: "a pipeline stage was never released",
                3: "the accumulator never completed", 4: "copies in flight did not land while winding down",
@@ -58,6 +58,7 @@ class TensorCoreKernels:
         self._latent = {}
         self._capped = {}
         self._ssd = {}
+        self._diff = {}
         # The weights that the products of a step stream, in launch order: recorded during one run
         # (``record_streams``) and replayed as hints during the next (``hint_streams``), so that every
         # few-token product asks for the weights of the product behind it to be brought into L2 while
@@ -359,6 +360,39 @@ class TensorCoreKernels:
         pairs = max(num_requests * kv_heads, 1)
         return max(1, min(296 // pairs, tiles // 2, 32))
 
+    # ------------------------------------------------------------------ differential attention
+    def differential_attention(self, q, k_pool, v_pool, block_table, b, out, scale, window, page_size, lam, out_scale, eps, gate,
+                               ws) -> bool:
+        """``CudaOps.differential_attention`` on the tensor cores; False where no such kernel takes the shape (widths that
+        are no multiple of 16 or beyond 128, groups of more than 64 heads)."""
+        T, Hq, D2 = q.shape
+        Hkv, vd, dim = k_pool.shape[1], v_pool.shape[3], D2 // 2
+        if dim % 16 or vd % 16 or dim > 128 or vd > 128 or Hq // Hkv > 64 or not scale > 0:
+            return False
+        lib = self._diff.get((dim, vd))
+        if lib is None:
+            lib = load_kernel_lib(diff_attention_lib_name(dim, vd))
+            lib.gb_last_error.restype = ctypes.c_char_p
+            lib.gb_diff_attention.argtypes = ([c_void_p] * 5 + [c_int] + [c_void_p] * 2 + [c_int] * 4 + [c_float] + [c_int] * 5
+                                              + [c_void_p, ctypes.c_longlong] + [c_float] * 3 + [c_void_p, ctypes.c_longlong, c_void_p])
+            lib.gb_diff_attention.restype = c_int
+            lib.gb_diff_attention_scratch_bytes.argtypes = [c_int, c_int, c_int]
+            lib.gb_diff_attention_scratch_bytes.restype = ctypes.c_longlong
+            self._diff[(dim, vd)] = lib
+        g, R = Hq // Hkv, b.num_requests
+        has_decode = b.min_q_len * g <= 16
+        splits = self.capped_plan(R, Hkv, b.max_kv_len, window, 0) if has_decode else 1
+        need = int(lib.gb_diff_attention_scratch_bytes(R, Hkv, splits))
+        scratch = (ws if ws is not None else self.ops.private_ws).get("diff_partials", (need,), torch.uint8) if need else None
+        code = lib.gb_diff_attention(
+            q.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), out.data_ptr(), block_table.data_ptr(), block_table.shape[1],
+            b.cu_q.data_ptr(), b.kv_lens.data_ptr(), T, R, Hq, Hkv, float(scale), int(window), int(page_size), int(b.max_q_len),
+            int(b.min_q_len), int(splits), None if scratch is None else scratch.data_ptr(), need, float(lam), float(out_scale),
+            float(eps), None if gate is None else gate.data_ptr(), gate.stride(0) if gate is not None else 0, self.ops._stream())
+        self.ops._check(lib, code, "diff_attention",
+                        ((2 if splits > 1 else 1) if has_decode else 0) + (1 if b.max_q_len * g > 16 else 0))
+        return True
+
     # ------------------------------------------------------------------ attention over cached latent rows
     @staticmethod
     def takes_latent(rank: int, rot: int) -> bool:
@@ -421,20 +455,22 @@ class TensorCoreKernels:
         """Sizes the kernel is compiled for: whole blocks of 16 of both, states that fit a CTA's registers."""
         return state_dim % 16 == 0 and head_dim % 16 == 0 and 16 <= state_dim <= 256 and head_dim >= 16
 
-    def ssd_chunk(self, act, step, skip, cu_q, slots, state, num_requests, heads, groups, state_dim, head_dim, y) -> bool:
+    def ssd_chunk(self, act, step, skip, cu_q, slots, state, num_requests, heads, groups, state_dim, head_dim, y,
+                  unit_state=None, unit_y=None) -> bool:
         """The recurrence of ``CudaOps.state_space`` from its prepared rows, chunk by chunk on the tensor
-        cores; False where the kernel does not take the sizes."""
+        cores; False where the kernel does not take the sizes. ``skip`` None: no skip term. ``unit_state`` (device address of
+        its place for head 0 in slot 0), ``unit_y [T, H]``: every head has one more row of state whose input is one."""
         if act.dtype != torch.bfloat16 or not self.takes_ssd(state_dim, head_dim):
             return False
         lib = self._ssd.get((state_dim, head_dim))
         if lib is None:
             lib = load_kernel_lib(ssd_lib_name(state_dim, head_dim))
             lib.gb_last_error.restype = ctypes.c_char_p
-            lib.gb_ssd_chunk.argtypes = [c_void_p] * 6 + [ctypes.c_longlong] + [c_int] * 3 + [c_void_p, c_void_p]
+            lib.gb_ssd_chunk.argtypes = [c_void_p] * 6 + [ctypes.c_longlong] + [c_int] * 3 + [c_void_p] * 4
             lib.gb_ssd_chunk.restype = c_int
             self._ssd[(state_dim, head_dim)] = lib
-        code = lib.gb_ssd_chunk(act.data_ptr(), step.data_ptr(), skip.data_ptr(), cu_q.data_ptr(), slots.data_ptr(),
+        code = lib.gb_ssd_chunk(act.data_ptr(), step.data_ptr(), None if skip is None else skip.data_ptr(), cu_q.data_ptr(), slots.data_ptr(),
                                 state.data_ptr(), state.stride(0), int(num_requests), int(heads), int(groups), y.data_ptr(),
-                                self.ops._stream())
+                                unit_state, None if unit_y is None else unit_y.data_ptr(), self.ops._stream())
         self.ops._check(lib, code, "ssd_chunk")
         return True

@@ -17,7 +17,7 @@ import torch
 
 from ..parts.base import (PartSpec, TensorSpec, PagedKV, PagedLatent, FixedState, LayerCache, build_part,
                           tensor_name, _REGISTRIES)
-from ..parts.block import BlockSpec
+from ..parts.block import BlockSpec, NormedInput
 
 
 @dataclass(frozen=True)
@@ -26,11 +26,13 @@ class LayerCall:
     ``reads_cache_of``: index of an earlier entry of the run order whose cache
     this call reads (it then stores nothing itself). A model that runs a stretch of its layers
     several times marks the first call of every pass: ``add_embedding`` adds the embedding's
-    output (the stream as it was before the first layer) to the stream before the call, and
-    ``add_row = (tensor, r)`` then adds row ``r`` of that model-level ``[rows, width]`` tensor."""
+    output (the stream as it was before the first layer) to the stream before the call, or
+    ``mix_embedding`` names a model-level ``[width, 2 width]`` matrix ``W`` and the stream becomes ``W [stream;
+    embedding's output]``; ``add_row = (tensor, r)`` then adds row ``r`` of that model-level ``[rows, width]`` tensor."""
     layer: int
     reads_cache_of: Optional[int] = None
     add_embedding: bool = False
+    mix_embedding: Optional[str] = None
     add_row: Optional[Tuple[str, int]] = None
 
 
@@ -47,12 +49,13 @@ class ModelSpec:
     head: Optional[str]                  # tensor name of the [vocab, width] head; None: tied
     embedding_init: Tuple = ("normal", 0.02)
     embedding_scale: float = 1.0         # the embedding's output is the table's row times this
+    embedding_norm: Optional[PartSpec] = None    # ... and then an RMS norm of it
     # the residual as several streams [T, streams, width], all equal to the embedding's output at the
     # start, summed before the final norm; None: one residual [T, width]
     streams: Optional[int] = None
     logit_scale: float = 1.0             # logits = head(x) * logit_scale ...
     logit_softcap: Optional[float] = None   # ... then c * tanh(logits / c)
-    # tensors of the model itself that no part owns (what ``LayerCall.add_row`` names): name -> spec
+    # tensors of the model itself that no part owns (what ``LayerCall.add_row`` and ``mix_embedding`` name): name -> spec
     extra_tensors: Optional[Dict[str, TensorSpec]] = None
     eos_token_ids: Tuple[int, ...] = ()  # generation ends on any of them (config.json may list several)
     # names a model folder may hold although the model reads nothing from them (a tied model's
@@ -77,6 +80,9 @@ class Decoder:
         self.spec = spec
         self.blocks = [_REGISTRIES["block"][b.arrangement](b) for b in spec.layers]
         self.final_norm = build_part("norm", spec.final_norm)
+        self.embedding_norm = build_part("norm", spec.embedding_norm) if spec.embedding_norm else None
+        if self.embedding_norm is not None and (not hasattr(self.embedding_norm, "fold") or spec.embedding_scale != 1.0 or spec.streams is not None):
+            raise ValueError("an embedding that is normed takes an RMS norm, no scale and one stream")
         self.ops = None
         self.dtype = None
         # cache needs of the run order
@@ -120,7 +126,7 @@ class Decoder:
     @property
     def graph_safe(self) -> bool:
         """Whether a decode step of this model may be captured in a CUDA graph: every part says so."""
-        return all(b.graph_safe for b in self.blocks) and self.final_norm.graph_safe
+        return all(b.graph_safe for b in self.blocks) and all(norm.graph_safe for norm, _ in self._model_norms())
 
     # ---- tensors ---------------------------------------------------------
     def expected_tensors(self) -> Dict[str, TensorSpec]:
@@ -130,12 +136,18 @@ class Decoder:
             for part, prefix in block.parts():
                 for local, ts in part.tensors().items():
                     out[tensor_name(prefix, local)] = ts
-        for local, ts in self.final_norm.tensors().items():
-            out[tensor_name(s.final_norm.prefix, local)] = ts
+        for norm, ns in self._model_norms():
+            for local, ts in norm.tensors().items():
+                out[tensor_name(ns.prefix, local)] = ts
         out.update(s.extra_tensors or {})
         if s.head is not None:
             out[s.head] = TensorSpec((s.vocab_size, s.width), init=s.embedding_init)
         return out
+
+    def _model_norms(self):
+        """The norms that belong to no layer, with their specs."""
+        pairs = [(self.final_norm, self.spec.final_norm), (self.embedding_norm, self.spec.embedding_norm)]
+        return [(norm, ns) for norm, ns in pairs if norm is not None]
 
     def load(self, tensors: Dict[str, torch.Tensor], ops, dtype: torch.dtype) -> None:
         """``tensors``: every name of ``expected_tensors()`` on the device."""
@@ -146,10 +158,13 @@ class Decoder:
         for block in self.blocks:
             for part, prefix in block.parts():
                 part.load({local: tensors[tensor_name(prefix, local)] for local in part.tensors()}, ops, dtype)
-        self.final_norm.load({local: tensors[tensor_name(s.final_norm.prefix, local)]
-                              for local in self.final_norm.tensors()}, ops, dtype)
-        self.extra = {name: tensors[name] for name in (s.extra_tensors or {})}
+        for norm, ns in self._model_norms():
+            norm.load({local: tensors[tensor_name(ns.prefix, local)] for local in norm.tensors()}, ops, dtype)
+        self.extra = {name: tensors[name].contiguous() for name in (s.extra_tensors or {})}
+        self.rows32 = {call.add_row: self.extra[call.add_row[0]][call.add_row[1]].float().contiguous()
+                       for call in s.order if call.add_row is not None}
         self.keeps_embedding = any(call.add_embedding for call in s.order)
+        self.mixes_embedding = any(call.mix_embedding is not None for call in s.order)
 
     # ---- one step ----------------------------------------------------------
     def forward(self, ctx, layer_caches: List[Optional[LayerCache]]) -> torch.Tensor:
@@ -160,10 +175,16 @@ class Decoder:
         if s.streams is not None:
             return self._forward_streams(ctx, layer_caches)
         x = ctx.ws.get("residual", (b.num_tokens, s.width), torch.float32)
-        if s.embedding_scale != 1.0:
+        # the operand [stream; embedding's output] of a mix, in the compute dtype
+        pair = ctx.ws.get("embedding_pair", (b.num_tokens, 2 * s.width), ctx.dtype) if self.mixes_embedding else None
+        if self.embedding_norm is not None:
+            ops.embedding_norm(self.embedding, b.token_ids, *self.embedding_norm.fold(), x, pair)
+        elif s.embedding_scale != 1.0:
             ops.embedding(self.embedding, b.token_ids, x, s.embedding_scale)
         else:
             ops.embedding(self.embedding, b.token_ids, x)
+        if pair is not None and self.embedding_norm is None:
+            ops.residual_norm(x, out=pair[:, s.width:])
         x0 = None
         if self.keeps_embedding:
             x0 = ctx.ws.get("embedding_out", (b.num_tokens, s.width), torch.float32)
@@ -172,12 +193,18 @@ class Decoder:
         pending = None
         for i, call in enumerate(s.order):
             block = self.blocks[call.layer]
-            if call.add_embedding or call.add_row is not None:
+            if call.mix_embedding is not None:
+                pending = self._mix_embedding(ctx, x, pair, call, block, rounded=pending is not None or (i == 0 and self.embedding_norm is not None))
+            elif call.add_embedding or call.add_row is not None:
                 row = self.extra[call.add_row[0]][call.add_row[1]] if call.add_row is not None else None
                 ops.residual_axpy(x, x0 if call.add_embedding else None, 1.0, row)
             nxt = self.blocks[s.order[i + 1].layer] if i + 1 < len(s.order) else None
-            takes = getattr(nxt, "takes_pending_norm", None)
-            next_norm = takes(ops) if takes is not None else None
+            if nxt is not None and s.order[i + 1].mix_embedding is not None:
+                # the mix in front of the next layer wants the stream rounded, beside the embedding's output
+                next_norm = NormedInput(out=pair[:, :s.width]) if getattr(block, "writes_normed_input", False) else None
+            else:
+                takes = getattr(nxt, "takes_pending_norm", None)
+                next_norm = takes(ops) if takes is not None else None
             if pending is not None or next_norm is not None:
                 pending = block.forward(ctx, x, layer_caches[i], pending=pending, next_norm=next_norm)
             else:
@@ -185,6 +212,24 @@ class Decoder:
             if ctx.layer_probe is not None:
                 ctx.layer_probe(i, x)
         return self._logits(ctx, x)
+
+    def _mix_embedding(self, ctx, x, pair, call, block, rounded):
+        """``x <- W [x; embedding's output] + row`` before a layer call. ``rounded``: the pass in front has left ``x``
+        in ``pair``. Returns the layer's normed input where the layer takes one from a pass over the residual."""
+        ops, width = self.ops, self.spec.width
+        if not rounded:
+            ops.residual_norm(x, out=pair[:, :width])
+        ops.linear(pair, self.extra[call.mix_embedding], x)
+        row = self.rows32.get(call.add_row)
+        takes = getattr(block, "takes_pending_norm", None)
+        wanted = takes(ops) if takes is not None else None
+        if isinstance(wanted, NormedInput):
+            weight, eps, out = wanted.into(ctx, x, 1)
+            ops.residual_norm(x, row=row, then_weight=weight, then_eps=eps, out=out)
+            return out
+        if row is not None:
+            ops.residual_axpy(x, None, 1.0, row)
+        return None
 
     def _logits(self, ctx, x) -> torch.Tensor:
         b, ops, s = ctx.batch, self.ops, self.spec
@@ -201,7 +246,7 @@ class Decoder:
         """The run order over a residual of several streams. A layer's last write to the streams
         computes the next layer's first normed input in the same pass where the kernels can."""
         b, ops, s = ctx.batch, self.ops, self.spec
-        if any(call.add_embedding or call.add_row is not None for call in s.order):
+        if any(call.add_embedding or call.mix_embedding is not None or call.add_row is not None for call in s.order):
             raise ValueError("a residual of several streams takes no additions between layer calls")
         x = ctx.ws.get("residual", (b.num_tokens, s.streams, s.width), torch.float32)
         ops.embedding(self.embedding, b.token_ids, x, s.embedding_scale)

@@ -38,6 +38,9 @@ class BlockSpec:
     feed_forward_gate: Optional[PartSpec] = None
     # for the arrangement that norms after the sum: x <- norm(post_alpha * x + part(x))
     post_alpha: float = 1.0
+    # for the arrangement with a norm in front of and behind each sublayer: the norms behind
+    mixer_post_norm: Optional[PartSpec] = None
+    feed_forward_post_norm: Optional[PartSpec] = None
 
 
 @register_block("pre_norm")
@@ -444,3 +447,84 @@ class ParallelBlock:
         self._run(ctx, ff, x, h, **kw)
         out, ctx.pending_norm = ctx.pending_norm, None
         return out
+
+
+class NormedInput:
+    """What a layer, or a step between layers, asks of the pass over the residual in front of it: the new
+    residual normed (``norm``, an RMS norm part) in the compute dtype, or with ``norm`` None just rounded to
+    it. ``out``: where it goes (a column range of a wider row will do); None: a buffer of the step's."""
+
+    def __init__(self, norm=None, out=None):
+        self.norm, self.out = norm, out
+
+    def into(self, ctx, x, turn):
+        """(weight or None, eps, destination)"""
+        out = self.out if self.out is not None else ctx.ws.get(f"normed_input_{turn}", tuple(x.shape), ctx.dtype)
+        weight, eps = self.norm.fold() if self.norm is not None else (None, 0.0)
+        return weight, eps, out
+
+
+@register_block("sandwich_norm")
+class SandwichNormBlock:
+    """A layer with a norm in front of and behind each sublayer: ``x <- x + norm1b(mixer(norm1(x)));
+    x <- x + norm2b(ffn(norm2(x)))``. The residual and a sublayer's output are 32-bit. What stands between two
+    sublayers' products is one pass over the row: the output's norm, the sum, and the norm that
+    the next sublayer reads (the next layer's, behind the last one)."""
+
+    #: its last pass writes what the next layer, or a step between layers, asks for (a ``NormedInput``)
+    writes_normed_input = True
+
+    def __init__(self, spec: BlockSpec):
+        if spec.residual_mult != 1.0 or spec.branches or spec.mixer_connection is not None or spec.mixer_gate is not None:
+            raise ValueError("a layer with norms on both sides of its sublayers takes no multiplier, branches, streams or gates")
+        self.spec = spec
+        build = lambda s: build_part("norm", s)
+        self.mixer, self.mixer_norm, self.mixer_post_norm = build_part("mixer", spec.mixer), build(spec.mixer_norm), build(spec.mixer_post_norm)
+        self.feed_forward = self.feed_forward_norm = self.feed_forward_post_norm = None
+        if spec.feed_forward:
+            self.feed_forward = build_part("feed_forward", spec.feed_forward)
+            self.feed_forward_norm, self.feed_forward_post_norm = build(spec.feed_forward_norm), build(spec.feed_forward_post_norm)
+        for norm in (self.mixer_norm, self.mixer_post_norm, self.feed_forward_norm, self.feed_forward_post_norm):
+            if norm is not None and not hasattr(norm, "fold"):
+                raise ValueError("a layer with norms on both sides of its sublayers takes RMS norms")
+
+    def parts(self):
+        s = self.spec
+        out = [(self.mixer_norm, s.mixer_norm.prefix), (self.mixer, s.mixer.prefix), (self.mixer_post_norm, s.mixer_post_norm.prefix)]
+        if self.feed_forward is not None:
+            out += [(self.feed_forward_norm, s.feed_forward_norm.prefix), (self.feed_forward, s.feed_forward.prefix),
+                    (self.feed_forward_post_norm, s.feed_forward_post_norm.prefix)]
+        return out
+
+    @property
+    def graph_safe(self):
+        return all(part.graph_safe for part, _ in self.parts())
+
+    def takes_pending_norm(self, ops):
+        """What the layer in front may leave for this one: its first norm, whole."""
+        return NormedInput(self.mixer_norm)
+
+    @staticmethod
+    def _join(ctx, x, y, norm, then, turn):
+        """``x += norm(y)``; ``then``: a ``NormedInput`` of the new ``x``, written in the same pass and returned."""
+        weight, eps = norm.fold()
+        if then is None:
+            ctx.ops.residual_norm(x, y, weight, eps)
+            return None
+        then_weight, then_eps, out = then.into(ctx, x, turn)
+        ctx.ops.residual_norm(x, y, weight, eps, then_weight=then_weight, then_eps=then_eps, out=out)
+        return out
+
+    def forward(self, ctx, x, cache, pending=None, next_norm=None):
+        """``pending``: this layer's normed input, written by the layer in front. ``next_norm``: what the next
+        layer said it takes; if that is a ``NormedInput``, the last pass writes it and it is returned."""
+        ctx.pending_norm = None
+        last = next_norm if isinstance(next_norm, NormedInput) else None
+        h = pending if pending is not None else self.mixer_norm.forward(ctx, x)
+        ff = self.feed_forward
+        # two buffers in turn: a sublayer's input may be read while the pass behind it writes the next one's
+        h2 = self._join(ctx, x, self.mixer.forward(ctx, h, cache), self.mixer_post_norm,
+                        NormedInput(self.feed_forward_norm) if ff is not None else last, 0 if ff is not None else 1)
+        if ff is None:
+            return h2
+        return self._join(ctx, x, ff.forward(ctx, h2), self.feed_forward_post_norm, last, 1)

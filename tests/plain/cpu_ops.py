@@ -80,7 +80,8 @@ class CpuOps:
             inv = torch.from_numpy(np.float32(1.0) / np.power(np.float32(rotary.theta),
                                                               np.float32(2.0) * i / np.float32(hd), dtype=np.float32))
         ang = positions.float()[:, None] * inv[None, :]
-        s, c = torch.sin(ang)[:, None, :], torch.cos(ang)[:, None, :]
+        factor = getattr(rotary, "factor", 1.0)
+        s, c = torch.sin(ang)[:, None, :] * factor, torch.cos(ang)[:, None, :] * factor
         out = torch.empty_like(v)
         if interleaved:
             a, b = v[..., 0::2], v[..., 1::2]
@@ -213,11 +214,20 @@ class CpuOps:
     def linear_gated(self, ctx, h, w_gate_up, act, kind="silu", limit=0.0):
         self.gated_act(h.float() @ w_gate_up.float().t(), act, kind, limit)
 
-    def route_topk(self, h, w_router, bias, top, ids, weights, score="softmax_chosen"):
+    def route_topk(self, h, w_router, bias, top, ids, weights, score="softmax_chosen", correction=None, groups=None):
         z = h.float() @ w_router.float().t()
         if bias is not None:
             z = z + bias.float()
-        order = torch.sort(-z, dim=-1, stable=True).indices[:, :top]
+        choice = z
+        if correction is not None:
+            choice = (torch.softmax(z, -1) if score == "softmax_all" else torch.sigmoid(z)) + correction
+        if groups is not None:              # only the best groups' experts (a group's score is its best expert's)
+            count, keep = groups
+            by_group = choice.reshape(choice.shape[0], count, -1)
+            best = torch.sort(-by_group.max(-1).values, dim=-1, stable=True).indices[:, :keep]
+            kept = torch.zeros(by_group.shape[:2], dtype=torch.bool).scatter_(1, best, True)
+            choice = torch.where(kept[:, :, None], by_group, torch.tensor(float("-inf"))).reshape(choice.shape)
+        order = torch.sort(-choice, dim=-1, stable=True).indices[:, :top]
         ids.copy_(order.to(torch.int32))
         chosen = torch.gather(z, 1, order)
         if score == "softmax_all":
@@ -230,16 +240,22 @@ class CpuOps:
         F = act.shape[2]
         for t in range(T):
             for j in range(top):
+                if int(ids[t, j]) >= w_gate_up.shape[0]:
+                    continue
                 x = h[t].float() * (float(in_scale[t, j]) if in_scale is not None else 1.0)
                 gu = (w_gate_up[int(ids[t, j])].float() @ x)[None, :]
                 self.gated_act(gu, act[t, j][None, :], kind, limit)
 
-    def moe_down(self, act, w_down, ids, weights, x, alpha=1.0):
+    def moe_down(self, act, w_down, ids, weights, x, alpha=1.0, identity=None):
         T, top, F = act.shape
         for t in range(T):
             total = torch.zeros(x.shape[1])
             for j in range(top):
                 wt = weights[t, j] if weights is not None else 1.0
+                if int(ids[t, j]) >= w_down.shape[0]:        # an expert that returns its input, or none
+                    if identity is not None:
+                        total += wt * identity[t].float()
+                    continue
                 total += wt * (w_down[int(ids[t, j])].float() @ act[t, j].float())
             x[t] += alpha * total
 
@@ -247,6 +263,8 @@ class CpuOps:
         """experts without a gate: act(up_e h), w_up [E, F, K]"""
         for t in range(h.shape[0]):
             for j, e in enumerate(ids[t].tolist()):
+                if e >= w_up.shape[0]:
+                    continue
                 u = w_up[e].float() @ h[t].float()
                 if in_scale is not None:
                     u = u * in_scale[t, j]
@@ -256,14 +274,14 @@ class CpuOps:
         return torch.stack([torch.cat([g, u], 0) for g, u in zip(gates, ups)]).contiguous()
 
     def routed_feed_forward(self, ctx, h, w_gate_up, w_down, ids, weights, x, kind, limit, alpha=1.0, scale_input=False,
-                            gated=True):
+                            gated=True, identity=False):
         T, top = ids.shape
         act = torch.zeros(T, top, w_down.shape[2], dtype=h.dtype)
         if gated:
             self.moe_gate_up(h, w_gate_up, ids, act, kind, limit, weights if scale_input else None)
         else:
             self.moe_up(h, w_gate_up, ids, act, kind, weights if scale_input else None)
-        self.moe_down(act, w_down, ids, None if scale_input else weights, x, alpha)
+        self.moe_down(act, w_down, ids, None if scale_input else weights, x, alpha, h if identity else None)
 
     # ---- a norm after the sum, gates per head, xIELU, a gated recurrence per channel, convolved projections ----
     def post_norm(self, x, y, alpha, weight, eps, row=None, rounded=None):
@@ -492,21 +510,25 @@ class CpuOps:
 
     # ---- normed queries and keys; sublayers whose outputs are normed ----
     def qk_norm_rope_append(self, src, cols, q_out, k_pool, v_pool, positions, token_req, block_table, heads, kv_heads,
-                            dim, vdim, q_weight, k_weight, eps, rotary, page_size, query_growth=None):
-        """queries and keys normed per head (weights 32-bit; None: not), rotated, queries (times 1 + coef
+                            dim, vdim, q_weight, k_weight, eps, rotary, page_size, query_growth=None, bias=None, maps=1):
+        """(bias over the columns q | k | v; maps neighbouring key heads lie in one row of the cache) queries and keys normed per head (weights 32-bit; None: not), rotated, queries (times 1 + coef
         ln(floor((p + 1) / every) + 1) at position p with query_growth = (coef, every)) out, keys and
         the untouched value columns into their pages; kv_heads 0: queries only"""
         T = src.shape[0]
         cq, ck, cv = cols
         q = src[:, cq:cq + heads * dim].float().reshape(T, heads, dim)
         k = src[:, ck:ck + kv_heads * dim].float().reshape(T, kv_heads, dim)
-        v = src[:, cv:cv + kv_heads * vdim].float().reshape(T, kv_heads, vdim)
+        v = src[:, cv:cv + kv_heads // maps * vdim].float().reshape(T, kv_heads // maps, vdim)
+        if bias is not None:
+            bq, bk, bv = torch.split(bias, [heads * dim, kv_heads * dim, kv_heads // maps * vdim])
+            q, k, v = q + bq.reshape(heads, dim), k + bk.reshape(kv_heads, dim), v + bv.reshape(-1, vdim)
         if q_weight is not None:
             q = q / torch.sqrt((q * q).mean(-1, keepdim=True) + eps) * q_weight.reshape(heads, dim)
         if k_weight is not None:
             k = k / torch.sqrt((k * k).mean(-1, keepdim=True) + eps) * k_weight
         if rotary is not None:
-            q, k = self._rotate(q, positions, rotary), self._rotate(k, positions, rotary)
+            n = rotary.head_dim          # the first n channels are turned
+            q, k = (torch.cat([self._rotate(u[..., :n], positions, rotary), u[..., n:]], -1) for u in (q, k))
         if query_growth is not None:
             coef, every = query_growth
             steps = torch.floor((positions.double() + 1.0) / every)
@@ -518,8 +540,81 @@ class CpuOps:
             pos = int(positions[t])
             page = int(block_table[int(token_req[t]), pos // page_size])
             if page >= 0:
-                k_pool[page, :, pos % page_size, :] = k[t].to(k_pool.dtype)
+                k_pool[page, :, pos % page_size, :] = k[t].reshape(kv_heads // maps, maps * dim).to(k_pool.dtype)
                 v_pool[page, :, pos % page_size, :] = v[t].to(v_pool.dtype)
+
+    # ---- norms on both sides, differential attention, a matrix memory ----
+    def residual_norm(self, x, y=None, weight=None, eps=0.0, row=None, then_weight=None, then_eps=0.0, out=None):
+        """x += rms(y) weight (or y) + row; out = rms(x) then_weight, or x, in out's dtype"""
+        def rms(v, e):
+            return v / torch.sqrt((v * v).mean(-1, keepdim=True) + e)
+        if y is not None:
+            x += rms(y, eps) * weight if weight is not None else y
+        if row is not None:
+            x += row
+        if out is not None:
+            out.copy_((rms(x, then_eps) * then_weight if then_weight is not None else x).to(out.dtype))
+
+    def embedding_norm(self, table, ids, weight, eps, x, pair=None):
+        """x = rms(table[ids]) weight; pair = [x; x] in its dtype"""
+        v = table[ids.long()].float()
+        x.copy_(v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps) * weight)
+        if pair is not None:
+            pair.copy_(torch.cat([x, x], -1).to(pair.dtype))
+
+    def differential_attention(self, ctx, q, k_pool, v_pool, block_table, out, scale, window, page_size, lam, out_scale, eps, gate):
+        """per head: the difference of two softmax maps over the same values, divided by its root mean square,
+        times out_scale and sigmoid(gate)"""
+        b = ctx.batch
+        T, H, D2 = q.shape
+        G, D, P = k_pool.shape[1], D2 // 2, v_pool.shape[3]
+        cu, lens = b.cu_q.tolist(), b.kv_lens.tolist()
+        for r in range(b.num_requests):
+            n = cu[r + 1] - cu[r]
+            for t in range(cu[r], cu[r + 1]):
+                pos = lens[r] - n + t - cu[r]
+                js = [j for j in range(max(0, pos + 1 - window) if window else 0, pos + 1) if int(block_table[r, j // page_size]) >= 0]
+                pages = block_table[r, torch.tensor(js) // page_size].long()
+                at = torch.tensor(js) % page_size
+                for h in range(H):
+                    k, v = k_pool[pages, h // (H // G), at].float(), v_pool[pages, h // (H // G), at].float()
+                    a = [torch.softmax((k[:, m * D:(m + 1) * D] @ q[t, h, m * D:(m + 1) * D].float()) * scale, 0) @ v for m in (0, 1)]
+                    o = a[0] - lam * a[1]
+                    o = o / torch.sqrt((o * o).mean() + eps) * out_scale
+                    if gate is not None:
+                        o = o * torch.sigmoid(gate[t, h])
+                    out[t, h * P:(h + 1) * P] = o.to(out.dtype)
+
+    def matrix_memory(self, ctx, act, gates, bias_i, bias_f, cap, norm_w, scale, eps, state, heads, dim, vdim, out):
+        """act: v | k | q (rounded to out's dtype), gates: output gate | input gate | forget gate; per request token by
+        token, the memory and its normalizer relative to the running maximum m"""
+        b = ctx.batch
+        H, D, P = heads, dim, vdim
+        HP, HD = H * P, H * D
+        act = act.to(out.dtype).float()
+        cu, slots = b.cu_q.tolist(), b.slots.tolist()
+        log_in = cap * torch.tanh((gates[:, HP:HP + H] + bias_i) / cap)
+        log_f = torch.nn.functional.logsigmoid(cap * torch.tanh((gates[:, HP + H:HP + 2 * H] + bias_f) / cap))
+        for r, slot in enumerate(slots):
+            if slot < 0:
+                out[cu[r]:cu[r + 1]] = 0
+                continue
+            S = state[slot, :HP * D].reshape(H, P, D).clone()
+            n = state[slot, HP * D:HP * D + HD].reshape(H, D).clone()
+            m = state[slot, HP * D + HD:HP * D + HD + H].clone()
+            for t in range(cu[r], cu[r + 1]):
+                v, k, q = (u.reshape(H, -1) for u in torch.split(act[t, :HP + 2 * HD], [HP, HD, HD]))
+                m2 = torch.maximum(log_f[t] + m, log_in[t])
+                keep, put, m = torch.exp(log_f[t] + m - m2), torch.exp(log_in[t] - m2), m2
+                S = keep[:, None, None] * S + put[:, None, None] * v[:, :, None] * k[:, None, :]
+                n = keep[:, None] * n + put[:, None] * k
+                o = torch.einsum("hpd,hd->hp", S, q) * scale
+                o = o / (torch.maximum((n * q).sum(-1).abs() * scale, torch.exp(-m)) + 1e-6)[:, None]
+                o = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps)
+                out[t] = (o.reshape(-1) * norm_w * torch.sigmoid(gates[t, :HP])).to(out.dtype)
+            state[slot, :HP * D] = S.reshape(-1)
+            state[slot, HP * D:HP * D + HD] = n.reshape(-1)
+            state[slot, HP * D + HD:HP * D + HD + H] = m
 
     @staticmethod
     def _unary(z, kind):
