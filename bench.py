@@ -9,6 +9,7 @@
     python bench.py --design luvapel [--size 2k,4k]     (the fourth, beside the third)
     python bench.py --design midulorn [--size 2k,4k]    (the fifth, beside the third)
     python bench.py --design fosovik [--size 2k,4k]     (the sixth, beside the third)
+    python bench.py --design ruvalix [--size 2k,4k]     (the seventh, beside the third)
     python bench.py --design kavenex [--size 2k,4k]     (a JSON line of its own: the second architecture
                                                          beside Llama at equal sizes, kernel beside like kernel)
 
@@ -1573,6 +1574,224 @@ def run_design_fosovik(args) -> dict:
     return out
 
 
+# ``--design ruvalix``: the Ruvalix design beside the Murilorn decoder (the closest of the engine's models: windowed
+# attention, a recurrence with a matrix of state per head, routed experts) at equal width, heads, value widths, window,
+# state sizes and depth (random weights). Four layers: attention, two matrix memories, attention, each with experts.
+RUVALIX_SIZES = {
+    "2k": dict(width=2048, heads=16, kv_heads=4, dim=64, vdim=128, window=1024, m_heads=4, m_dim=256, m_vdim=512, experts=16, identity=4,
+               groups=4, keep=2, top=4, expert_ff=1408, shared_ff=1408, vocab=32000, d_heads=32, d_kv_heads=16, d_dim=128, d_vdim=128, rank=64),
+    "4k": dict(width=4096, heads=32, kv_heads=8, dim=64, vdim=128, window=1024, m_heads=8, m_dim=256, m_vdim=512, experts=16, identity=4,
+               groups=4, keep=2, top=4, expert_ff=2752, shared_ff=2752, vocab=32000, d_heads=64, d_kv_heads=16, d_dim=128, d_vdim=128, rank=128),
+}
+
+
+def ruvalix_configs(z):
+    moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"], "identity": z["identity"], "groups": {"count": z["groups"], "keep": z["keep"]}},
+           "expert": {"ff": z["expert_ff"]}, "shared": {"ff": z["shared_ff"]}}
+    att = {"type": "attention", "mlp": moe, "mixer": {
+        "heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5, "diff": 0.6,
+        "mask": {"size": z["window"]}, "rot": {"base": 500000.0, "dims": z["dim"] // 2, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}}
+    mem = {"type": "mlstm", "mlp": moe, "mixer": {"heads": z["m_heads"], "dim": z["m_dim"], "vdim": z["m_vdim"], "gate_cap": 15.0}}
+    ruvalix = {"architecture": "Ruvalix", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "max_positions": 4096,
+               "layers": [att, mem, mem, att]}
+    moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["expert_ff"]}}
+    attn = {"type": "attention", "mixer": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": 2 * z["dim"], "vdim": z["vdim"],
+                                           "scale": (2 * z["dim"]) ** -0.5, "softcap": 30.0, "mask": {"size": z["window"], "keep_first": 4}}}
+    delta = {"type": "channel_delta", "mixer": {"heads": z["d_heads"], "kv_heads": z["d_kv_heads"], "dim": z["d_dim"],
+                                                "vdim": z["d_vdim"], "conv": 4, "decay_rank": z["rank"], "gate_rank": z["rank"]}}
+    murilorn = {"architecture": "Murilorn", "vocab": z["vocab"], "width": z["width"], "embedding": {"scale": 1.0},
+                "norm": {"eps": 1e-5}, "streams": 2, "logit_scale": 1.0, "logit_softcap": 30.0, "max_positions": 4096,
+                "layers": [dict(m, mlp=moe) for m in (attn, delta, delta, attn)]}
+    return ruvalix, murilorn
+
+
+def run_design_ruvalix(args) -> dict:
+    """Prefill and decode throughput of the Ruvalix design and of the Murilorn decoder at equal sizes, and
+    the design's kernels beside the like kernels of the engine's other models, each against its roofline (the
+    slower of bytes / measured copy rate and FLOPs / measured bfloat16 rate)."""
+    import numpy as np
+    import torch
+    from types import SimpleNamespace
+    from garuda_b200 import Engine, StepEntry
+    from garuda_b200.engine.batch import Workspace
+    from garuda_b200.parts.rotary import Rotary
+    from garuda_b200.weights import write_random_model
+
+    hbm_peak, tflops_peak, peak_kind = peaks()
+    ev = lambda: torch.cuda.Event(enable_timing=True)
+    dev = torch.device("cuda:0")
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+
+    def timed(fn, reps=10):
+        for _ in range(3):
+            fn()
+        times = []
+        for _ in range(reps):
+            flush.zero_()
+            s, e = ev(), ev()
+            torch.cuda.synchronize()
+            s.record()
+            fn()
+            e.record()
+            torch.cuda.synchronize()
+            times.append(s.elapsed_time(e))
+        return sorted(times)[len(times) // 2]
+
+    def roof(ms, flops=0.0, nbytes=0.0):
+        ideal = max(flops / (tflops_peak * 1e12), nbytes / (hbm_peak * 1e9)) * 1e3
+        return {"ms": round(ms, 4), "roofline_ms": round(ideal, 4), "frac": round(ideal / ms, 4)}
+
+    out = {"design": "ruvalix", "beside": "murilorn", "peaks": peak_kind, "hbm_gbs": hbm_peak, "bf16_tflops": tflops_peak,
+           "dtype": "bf16", "data": "synthetic",
+           "timing": "CUDA events, 3 warm-up runs, L2 flushed before every timed run, median", "sizes": {}}
+    B, CTX, T = 8, 2048, PREFILL_TOKENS
+    for name in (args.size.split(",") if args.size else list(RUVALIX_SIZES)):
+        z = RUVALIX_SIZES[name]
+        rec, engines = {}, {}
+        for arch, cfg in zip(("ruvalix", "murilorn"), ruvalix_configs(z)):
+            if args.only == "attention" or (args.only and arch == "murilorn"):
+                continue
+            tmp = tempfile.mkdtemp(prefix="garuda_bench_", dir="/dev/shm" if os.path.isdir("/dev/shm") else None)
+            try:
+                write_random_model(tmp, cfg, seed=0, store_dtype=torch.bfloat16)
+                engine = Engine(tmp, dtype="bfloat16", context=4096, page_size=32, kv_tokens=B * CTX + 4096 + 64,
+                                max_concurrent=B, max_batch_tokens=T, prefill_chunk=T, ignore_eos=True)
+            finally:
+                shutil.rmtree(tmp, ignore_errors=True)
+            engines[arch] = engine
+            runner, rng, V = engine.runner, np.random.default_rng(0), z["vocab"]
+            toks = rng.integers(0, V, T).tolist()
+            rid = [0]
+
+            def prefill():
+                rid[0] += 1
+                runner.run([StepEntry(10_000 + rid[0], toks, [T - 1])])
+                runner.end(10_000 + rid[0])
+
+            rec[arch] = {}
+            if args.only != "decode":
+                ms = timed(prefill, reps=5)
+                rec[arch] = {"prefill_2048_ms": round(ms, 3), "prefill_tok_s": round(T / ms * 1e3)}
+            if args.only != "prefill":
+                steps = 48
+                for r in range(B):
+                    runner.run([StepEntry(r, rng.integers(0, V, CTX - steps - 8).tolist(), [])])
+                feed = rng.integers(0, V, (steps + 8, B))
+                for i in range(8):
+                    runner.run([StepEntry(r, [int(feed[i, r])], [0]) for r in range(B)])
+                marks = [ev() for _ in range(steps + 1)]
+                torch.cuda.synchronize()
+                marks[0].record()
+                for i in range(steps):
+                    runner.run([StepEntry(r, [int(feed[8 + i, r])], [0]) for r in range(B)])
+                    marks[i + 1].record()
+                torch.cuda.synchronize()
+                each = sorted(marks[i].elapsed_time(marks[i + 1]) for i in range(steps))
+                for r in range(B):
+                    runner.end(r)
+                rec[arch].update({"decode_b8_ctx2048_ms": round(each[len(each) // 2], 4),
+                                  "decode_tok_s": round(B / each[len(each) // 2] * 1e3),
+                                  "graph_replays": runner.graphs.replays,
+                                  "kernels_per_decode_step": runner.graphs.launches_replayed(B)})
+            if engine.ops.tc is not None:
+                engine.ops.tc.check_errors()
+        if args.only:
+            out["sizes"][name] = rec
+            continue
+        # ------------------------------------------------------------ kernel beside like kernel
+        ops = engines["ruvalix"].ops
+        bf = torch.bfloat16
+        H, Hkv, hd, vd, W, ps, win = z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["width"], 32, z["window"]
+        ctx = SimpleNamespace(ws=Workspace(dev), step_cache={})
+        ws, kern = ctx.ws, {}
+        vec = lambda m, s=1.0: torch.randn(m, device=dev) * s
+        rotary = Rotary(500000.0, hd // 2, scaling=dict(factor=4.0, original=8192, fast=32.0, slow=1.0)).rotary
+        for label, nreq, q_len, kv_len in (("prefill_2048", 1, T, T), ("decode_b8_ctx2048", B, 1, CTX)):
+            pages, n = (kv_len + ps - 1) // ps, nreq * q_len
+            bt = torch.arange(nreq * pages, dtype=torch.int32, device=dev).view(nreq, pages)
+            cu = torch.arange(nreq + 1, dtype=torch.int32, device=dev) * q_len
+            kvl = torch.full((nreq,), kv_len, dtype=torch.int32, device=dev)
+            req = torch.arange(nreq, dtype=torch.int32, device=dev).repeat_interleave(q_len)
+            pos = (torch.arange(q_len, dtype=torch.int32, device=dev) + (kv_len - q_len)).repeat(nreq)
+            ctx.batch = SimpleNamespace(cu_q=cu, token_req=req, positions=pos, kv_lens=kvl, num_requests=nreq, max_q_len=q_len,
+                                        min_q_len=q_len, max_kv_len=kv_len, slots=torch.arange(nreq, dtype=torch.int32, device=dev))
+            # two maps over the same values, beside Murilorn's capped attention whose keys are as wide as both maps
+            q = torch.randn(n, H, 2 * hd, device=dev).to(bf)
+            kp, vp = torch.randn(nreq * pages, Hkv, ps, 2 * hd, device=dev).to(bf), torch.randn(nreq * pages, Hkv, ps, vd, device=dev).to(bf)
+            o, gate = torch.empty(n, H * vd, dtype=bf, device=dev), vec(n * H).view(n, H)
+            keys = nreq * sum(min(i, win) for i in range(kv_len - q_len + 1, kv_len + 1))
+            moved = 2.0 * (nreq * min(kv_len, win + q_len) * Hkv * (2 * hd + vd) + q.numel() + o.numel())
+            kern[f"differential_attention_{label}"] = roof(timed(lambda: ops.differential_attention(
+                ctx, q, kp, vp, bt, o, hd ** -0.5, win, ps, 0.7, 0.4, 1e-5, gate)), 2.0 * H * (2 * hd + 2 * vd) * keys, moved)
+            args_a = (q, kp, vp, bt, cu, kvl, req, o, (2 * hd) ** -0.5, win, ps, nreq, q_len, kv_len)
+            kern[f"murilorn_capped_sink_attention_{label}"] = roof(
+                timed(lambda: ops.paged_attention(*args_a, ws=ws, min_q_len=q_len, softcap=30.0, sink=True, keep_first=4)),
+                2.0 * H * (2 * hd + vd) * keys, moved)
+            # the projected row into queries and pages: biased, normed and rotated here, biased there
+            cols = 2 * (H + Hkv) * hd + Hkv * vd
+            row, bias = vec(n * cols).view(n, cols), vec(cols)
+            qw, kw = torch.ones(2 * H, hd, device=dev), torch.ones(hd, device=dev)
+            kern[f"bias_norm_rotate_store_{label}"] = roof(timed(lambda: ops.qk_norm_rope_append(
+                row, (0, 2 * H * hd, 2 * (H + Hkv) * hd), q.view(n, 2 * H, hd), kp, vp, pos, req, bt, 2 * H, 2 * Hkv, hd, vd, qw, kw, 1e-5, rotary, ps,
+                bias=bias, maps=2)), 0, 6.0 * row.numel())
+            kern[f"murilorn_bias_store_{label}"] = roof(
+                timed(lambda: ops.qkv_bias_append(row, bias, q, kp, vp, pos, req, bt, H, Hkv, 2 * hd, vd, ps)), 0, 6.0 * row.numel())
+            # the recurrences, everything between the projections: bytes are the rows in and out and the state
+            MH, MD, MP = z["m_heads"], z["m_dim"], z["m_vdim"]
+            inner, C = MH * MP, MH * (MP + 2 * MD)
+            act = vec(n * C).view(n, C).to(torch.float32 if q_len == 1 else bf)
+            gates, nw, so = vec(n * (inner + 2 * MH)).view(n, -1), vec(inner), torch.empty(n, inner, dtype=bf, device=dev)
+            st = torch.zeros(nreq, (inner * MD + MH * MD + MH + 3) // 4 * 4, device=dev)
+            b_i, b_f = vec(MH), vec(MH) + 4.0
+            ms = timed(lambda: ops.matrix_memory(ctx, act, gates, b_i, b_f, 15.0, nw, MD ** -0.5, 1e-5, st, MH, MD, MP, so))
+            kern[f"matrix_memory_{label}"] = roof(ms, 0, act.numel() * act.element_size() + 4.0 * gates.numel() + 2.0 * so.numel() + 2 * 4.0 * st.numel())
+            dH, dG, dd, dv, taps = z["d_heads"], z["d_kv_heads"], z["d_dim"], z["d_vdim"], 4
+            DC = 2 * dG * dd + dH * dv
+            conv_w, a_log, dnw = torch.randn(DC, taps, device=dev) * 0.3, vec(dH, 0.3), torch.ones(dv, device=dev)
+            dstate = torch.zeros(nreq, dH * dd * dv + (taps - 1) * DC, device=dev)
+            dproj, second = torch.randn(n, DC + dH, device=dev), torch.randn(n, dH * dd + dH * dv, device=dev)
+            ddt, do = vec(dH * dd), torch.empty(n, dH * dv, dtype=bf, device=dev)
+            ms = timed(lambda: ops.delta_rule(ctx, dproj, second, conv_w, a_log, ddt, dnw, 1e-5, dstate, dH, dG, dd, dv, taps, do))
+            kern[f"murilorn_channel_delta_rule_{label}"] = roof(ms, 0, 4.0 * (dproj.numel() + second.numel()) + 2.0 * do.numel()
+                                                                + 2 * 4.0 * dstate.numel())
+            del q, kp, vp, o, row, act, gates, so, dproj, second, do
+        # experts, a part of whose choices return their input, beside experts that all compute; the choice itself; what
+        # stands between two sublayers, beside Luvapel's pass over the row and Llama's norm
+        E, I, top, EF = z["experts"], z["identity"], z["top"], z["expert_ff"]
+        mat = lambda *s: (torch.randn(*s, device=dev) * 0.02).to(bf)
+        gu = ops.pack_expert_gate_up([mat(EF, W) for _ in range(E)], [mat(EF, W) for _ in range(E)])
+        down, router, corr = mat(E, W, EF), mat(E + I, W), vec(E + I, 0.01)
+        wv, wv2 = vec(W, 0.1) + 1.0, vec(W, 0.1) + 1.0
+        for label, M in (("2048_tokens", T), ("8_tokens", B)):
+            h, x = torch.randn(M, W, device=dev).to(bf), torch.zeros(M, W, device=dev)
+            wts = torch.rand(M, top, device=dev)
+            for what, choices, kw in (("identity_experts", E + I, {"identity": True}), ("murilorn_gated_experts", E, {})):
+                ids = torch.stack([torch.randperm(choices, device=dev)[:top] for _ in range(M)]).to(torch.int32)
+                real = int((ids < E).sum())
+                used = len(torch.unique(ids[ids < E]))
+                ms = timed(lambda: ops.routed_feed_forward(ctx, h, gu, down, ids, wts, x, "silu", 0.0, **kw))
+                kern[f"{what}_{label}"] = roof(ms, 2.0 * real * 3 * EF * W, 2.0 * used * 3 * EF * W)
+            ids = torch.empty(M, top, dtype=torch.int32, device=dev)
+            cost = (2.0 * M * (E + I) * W, 2.0 * (h.numel() + router.numel()))
+            kern[f"choice_in_groups_{label}"] = roof(timed(lambda: ops.route_topk(
+                h, router, None, top, ids, wts, score="softmax_all", correction=corr, groups=(z["groups"], z["keep"]))), *cost)
+            kern[f"murilorn_choice_{label}"] = roof(timed(lambda: ops.route_topk(h, router, None, top, ids, wts, score="sigmoid")), *cost)
+            y, hb = torch.randn(M, W, device=dev), torch.empty(M, W, dtype=bf, device=dev)
+            kern[f"residual_norm_{label}"] = roof(timed(lambda: ops.residual_norm(x, y, wv, 1e-5, then_weight=wv2, then_eps=1e-5, out=hb)), 0, 14.0 * M * W)
+            kern[f"luvapel_sublayer_merge_{label}"] = roof(timed(lambda: ops.sublayer_merge([y], None, 1e-5, x=x, weight=wv, rounded=hb)), 0, 14.0 * M * W)
+            kern[f"llama_rms_norm_{label}"] = roof(timed(lambda: ops.rmsnorm(x, wv, 1e-5, hb)), 0, 6.0 * M * W)
+            table, tok = mat(z["vocab"], W), torch.randint(0, z["vocab"], (M,), dtype=torch.int32, device=dev)
+            kern[f"embedding_norm_{label}"] = roof(timed(lambda: ops.embedding_norm(table, tok, wv, 1e-5, x)), 0, 6.0 * M * W)
+            kern[f"llama_embedding_{label}"] = roof(timed(lambda: ops.embedding(table, tok, x)), 0, 6.0 * M * W)
+            del table
+        rec["kernels"] = kern
+        rec["config"] = {k: v for k, v in z.items()}
+        out["sizes"][name] = rec
+        del engines
+        torch.cuda.empty_cache()
+    return out
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1587,8 +1806,8 @@ def main() -> int:
     ap.add_argument("--context", type=int, default=0, help="context reached with --only decode (default: the shape's); keys with --only attention")
     ap.add_argument("--layers", type=int, default=0,
                     help="fewer layers than the configuration has (reported beside the full number)")
-    ap.add_argument("--design", choices=["kavenex", "murilorn", "luvapel", "midulorn", "fosovik"],
-                    help="instead of the default workload: this design beside the Llama decoder (luvapel, midulorn and fosovik: "
+    ap.add_argument("--design", choices=["kavenex", "murilorn", "luvapel", "midulorn", "fosovik", "ruvalix"],
+                    help="instead of the default workload: this design beside the Llama decoder (luvapel, midulorn, fosovik and ruvalix: "
                          "beside Murilorn, the closest of the engine's models) at equal sizes")
     ap.add_argument("--size", default="", help="with --design: which of its sizes (2k, 4k; default both)")
     args = ap.parse_args()
@@ -1607,7 +1826,7 @@ def main() -> int:
         return 2
     if args.design:
         run = {"murilorn": run_design_murilorn, "luvapel": run_design_luvapel, "kavenex": run_design,
-               "midulorn": run_design_midulorn, "fosovik": run_design_fosovik}[args.design]
+               "midulorn": run_design_midulorn, "fosovik": run_design_fosovik, "ruvalix": run_design_ruvalix}[args.design]
         print(json.dumps(run(args)))
         return 0
     print(json.dumps(run_ours(args)))

@@ -576,14 +576,15 @@ class CpuOps:
                 js = [j for j in range(max(0, pos + 1 - window) if window else 0, pos + 1) if int(block_table[r, j // page_size]) >= 0]
                 pages = block_table[r, torch.tensor(js) // page_size].long()
                 at = torch.tensor(js) % page_size
-                for h in range(H):
-                    k, v = k_pool[pages, h // (H // G), at].float(), v_pool[pages, h // (H // G), at].float()
-                    a = [torch.softmax((k[:, m * D:(m + 1) * D] @ q[t, h, m * D:(m + 1) * D].float()) * scale, 0) @ v for m in (0, 1)]
-                    o = a[0] - lam * a[1]
-                    o = o / torch.sqrt((o * o).mean() + eps) * out_scale
-                    if gate is not None:
-                        o = o * torch.sigmoid(gate[t, h])
-                    out[t, h * P:(h + 1) * P] = o.to(out.dtype)
+                k = k_pool[pages, :, at].float().repeat_interleave(H // G, 1)          # [keys, H, 2 D]
+                v = v_pool[pages, :, at].float().repeat_interleave(H // G, 1)
+                a = [torch.einsum("jh,jhp->hp", torch.softmax(torch.einsum("jhd,hd->jh", k[..., m * D:(m + 1) * D], q[t, :, m * D:(m + 1) * D].float())
+                                                              * scale, 0), v) for m in (0, 1)]
+                o = a[0] - lam * a[1]
+                o = o / torch.sqrt((o * o).mean(-1, keepdim=True) + eps) * out_scale
+                if gate is not None:
+                    o = o * torch.sigmoid(gate[t])[:, None]
+                out[t] = o.reshape(-1).to(out.dtype)
 
     def matrix_memory(self, ctx, act, gates, bias_i, bias_f, cap, norm_w, scale, eps, state, heads, dim, vdim, out):
         """act: v | k | q (rounded to out's dtype), gates: output gate | input gate | forget gate; per request token by
