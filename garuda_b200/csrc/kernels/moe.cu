@@ -16,27 +16,32 @@ constexpr int MAX_TOP = 32;
 // descending order (the lower index first among equals); weights = softmax over the chosen logits
 // (mode 0), or each chosen expert's own sigmoid(z_e), not renormalized (mode 1), or its share of a
 // softmax over all E logits, not renormalized either (mode 2).
+// logits [T, E] (or null): h . W is in there already, the block is one warp.
 // correction [E] (or null; modes 1 and 2): the choice is by score + correction, the weights are the scores
 // without it. groups > 0: the experts form so many equal groups of neighbours, a group's score is its best
 // expert's, and only experts of the `keep` best groups (the lower index first among equals) can be chosen.
 template <typename HT, typename WT>
 __global__ void __launch_bounds__(256)
-route_topk_kernel(const HT* __restrict__ h, const WT* __restrict__ w, const float* __restrict__ bias, int T, int E,
-                  int K, int top, int mode, const float* __restrict__ correction, int groups, int keep,
+route_topk_kernel(const HT* __restrict__ h, const WT* __restrict__ w, const float* __restrict__ logits,
+                  const float* __restrict__ bias, int T, int E, int K, int top, int mode, const float* __restrict__ correction, int groups, int keep,
                   int32_t* __restrict__ ids, float* __restrict__ weights) {
   gb::pdl_launch_dependents();
   gb::pdl_wait();
   extern __shared__ __align__(16) float sm[];        // h[K], z[E] (what the choice goes by), score[E], best of each group[E]
   float* h_s = sm;
-  float* z = sm + K;
+  float* z = sm + (logits != nullptr ? 0 : K);
   float* score = z + E;
   float* best_of = score + E;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   const int t = blockIdx.x;
   const HT* hr = h + (size_t)t * K;
-  for (int k = threadIdx.x; k < K; k += blockDim.x) h_s[k] = gb::to_float<HT>(hr[k]);
+  if (logits != nullptr) {
+    for (int e = threadIdx.x; e < E; e += blockDim.x) z[e] = logits[(size_t)t * E + e] + (bias ? bias[e] : 0.f);
+  } else {
+    for (int k = threadIdx.x; k < K; k += blockDim.x) h_s[k] = gb::to_float<HT>(hr[k]);
+  }
   __syncthreads();
-  for (int e = warp; e < E; e += warps) {
+  for (int e = warp; e < (logits != nullptr ? 0 : E); e += warps) {
     const WT* wr = w + (size_t)e * K;
     float acc = 0.f;
     if (sizeof(WT) == 2 && K % 8 == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0) {        // eight neighbouring weights in one load (rows start on 16 bytes)
@@ -243,7 +248,8 @@ moe_down_kernel(const AT* __restrict__ act, const WT* __restrict__ w, const int3
 
 }  // namespace
 
-GB_EXPORT int gb_route_topk(const void* h, int h_dtype, const void* w, const float* bias, int w_dtype, int T, int E,
+// logits [T, E] 32-bit (or null): the products h . W, made by the caller.
+GB_EXPORT int gb_route_topk(const void* h, int h_dtype, const void* w, const float* logits, const float* bias, int w_dtype, int T, int E,
                             int K, int top, int mode, const float* correction, int groups, int keep, int32_t* ids,
                             float* weights, cudaStream_t stream) {
   if (T <= 0) return GB_OK;
@@ -253,7 +259,7 @@ GB_EXPORT int gb_route_topk(const void* h, int h_dtype, const void* w, const flo
   if (correction != nullptr && mode == 0) return gb::fail(GB_BAD_ARGUMENT, "route_topk: a correction goes with scores of their own");
   if (groups < 0 || (groups > 0 && (E % groups || keep < 1 || keep > groups || top > E / groups * keep)))
     return gb::fail(GB_BAD_ARGUMENT, "route_topk: %d of %d groups of %d experts, %d chosen", keep, groups, E, top);
-  const size_t smem = (size_t)(3 * E + K) * sizeof(float);
+  const size_t smem = (size_t)(3 * E + (logits != nullptr ? 0 : K)) * sizeof(float);
   if (smem > 200 * 1024) return gb::fail(GB_UNSUPPORTED, "route_topk: width %d", K);
   return GB_DISPATCH_DTYPE(h_dtype, HT, [&]() -> int {
     return GB_DISPATCH_DTYPE(w_dtype, WT, [&]() -> int {
@@ -262,8 +268,8 @@ GB_EXPORT int gb_route_topk(const void* h, int h_dtype, const void* w, const flo
         if (e != cudaSuccess) return gb::fail(GB_CUDA_ERROR, "route_topk: %s", cudaGetErrorString(e));
       }
       return gb::check_pdl_launch(
-          gb::launch_pdl(route_topk_kernel<HT, WT>, dim3(T), dim3(256), smem, stream,
-                         dim3(1, 1, 1), (const HT*)h, (const WT*)w, bias, T, E, K, top, mode, correction, groups, keep, ids, weights),
+          gb::launch_pdl(route_topk_kernel<HT, WT>, dim3(T), dim3(logits != nullptr ? 32 : 256), smem, stream,
+                         dim3(1, 1, 1), (const HT*)h, (const WT*)w, logits, bias, T, E, K, top, mode, correction, groups, keep, ids, weights),
           "route_topk");
     });
   });

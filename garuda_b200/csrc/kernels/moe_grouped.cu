@@ -286,6 +286,7 @@ GB_EXPORT long long gb_moe_grouped_index_words(long long R, int E) {
 // h [T, K], w_gate_up by layout: 0 [E, 2F, K] (gate rows, then up rows), 1 [E, 128 * ceil(F / 64), K] (gate and up
 // rows in groups of 64), 2 [E, F, K] (experts without a gate: act(up h), kind as for gb_moe_up),
 // w_down [E, N, F] bfloat16; ids [T, top], weights [T, top]; x [T, N] 32-bit.
+// x null: nothing is added up, the pairs' rows are left in y and their numbers (pair -> row, -1: none) in index + T * top.
 // index: gb_moe_grouped_index_words int32; act: [T * top, F] bfloat16; y: [T * top, N] 32-bit.
 GB_EXPORT int gb_moe_grouped(const void* h, const void* w_gate_up, const void* w_down, const int32_t* ids,
                              const float* weights, float* x, int T, int top, int E, int F, int K, int N, int kind,
@@ -344,7 +345,7 @@ GB_EXPORT int gb_moe_grouped(const void* h, const void* w_gate_up, const void* w
   else
     rc = launch_grouped<1, 4, 1, 1, PLAIN, float>(grid_n, stream, "moe_down_grouped", ac, F, zero, none, 1, wd, d_group, y, N,
                                                  zero, N, F, te, t0, tr, nt, 0, 0, 0.f, 0, no_scale);
-  if (rc != GB_OK) return rc;
+  if (rc != GB_OK || x == nullptr) return rc;
   moe_combine_kernel<<<combine_grid(T, N), 256, 0, stream>>>(y, pair_row, out_weights, x, top, N, alpha,
                                             TanhNorm{(__nv_bfloat16*)norm_out, norm_w, norm_b, norm_alpha}, identity ? hh : nullptr);
   return gb::check_launch("moe_combine");

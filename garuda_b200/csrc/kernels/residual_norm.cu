@@ -1,7 +1,9 @@
 // What stands between two sublayers' products in a layer with norms in front of and behind each sublayer, as one
 // pass over the residual's row; and the normed embedding such a model starts from. 32-bit arithmetic.
 //
-//   residual_norm    x <- x + rms(y) * w_y (or + y, or nothing) + row;   out = rms(x) * w_out, or x, in out's dtype
+//   residual_norm    x <- x + rms(y) * w_y (or + y, or nothing) + row;   out = rms(x) * w_out, or x, in out's dtype;
+//                    y may be what routed experts leave for it: a row per (token, choice) pair, summed with the
+//                    choices' weights as it is read
 //   embedding_norm   x = rms(table[id]) * w;   pair = [x | x] in its dtype (the operand of a product that mixes the
 //                    stream with the embedding's output: its first half is written again before every mix)
 #include <type_traits>
@@ -42,6 +44,13 @@ struct NormStep {
   float y_eps, out_eps;
   long long out_stride;
   int d;
+  // routed experts' rows, added to y: sum_j weights[t][j] * rows[pair_row[t top + j]], j in the router's order; a pair without a row
+  // stands for identity[t] (null: nothing). top 0: none.
+  const float* rows;         // [., d]
+  const int32_t* pair_row;
+  const float* weights;      // [T, top]
+  const __nv_bfloat16* identity;
+  int top;
 };
 
 // One block per token; a thread keeps PER groups of four neighbouring channels of the row in registers from the
@@ -72,18 +81,40 @@ residual_norm_kernel(const NormStep p, OT* __restrict__ out) {
     for (int j = 0; j < 4; ++j) x[k][j] = 0.f;
     if (c < d) load4(xr, c, x[k]);
   }
-  if (p.y != nullptr) {
-    const float* yr = p.y + t * d;
+  const bool adds = p.y != nullptr || p.top > 0;
+  if (adds) {
     float y[PER][4], ss = 0.f;
 #pragma unroll
     for (int k = 0; k < PER; ++k) {
       const int c = (threadIdx.x + k * blockDim.x) * 4;
 #pragma unroll
       for (int j = 0; j < 4; ++j) y[k][j] = 0.f;
-      if (c < d) load4(yr, c, y[k]);
+      if (c < d && p.y != nullptr) load4(p.y + t * d, c, y[k]);
+    }
+#pragma unroll 2
+    for (int e = 0; e < p.top; ++e) {
+      const int from = p.pair_row[t * p.top + e];
+      const float wt = p.weights[t * p.top + e];
+#pragma unroll
+      for (int k = 0; k < PER; ++k) {
+        const int c = (threadIdx.x + k * blockDim.x) * 4;
+        if (c >= d) continue;
+        float v[4] = {0.f, 0.f, 0.f, 0.f};
+        if (from >= 0) {
+          load4(p.rows + (size_t)from * d, c, v);
+        } else if (p.identity != nullptr) {
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            if (VEC || c + j < d) v[j] = __bfloat162float(p.identity[t * d + c + j]);
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) y[k][j] = fmaf(wt, v[j], y[k][j]);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < PER; ++k)
 #pragma unroll
       for (int j = 0; j < 4; ++j) ss = fmaf(y[k][j], y[k][j], ss);
-    }
     const float inv = p.y_w != nullptr ? 1.0f / sqrtf(block_sum(ss, red) / (float)d + p.y_eps) : 1.0f;
 #pragma unroll
     for (int k = 0; k < PER; ++k) {
@@ -105,7 +136,7 @@ residual_norm_kernel(const NormStep p, OT* __restrict__ out) {
       for (int j = 0; j < 4; ++j) x[k][j] += r[j];
     }
   }
-  if (p.y != nullptr || p.row != nullptr) {
+  if (adds || p.row != nullptr) {
 #pragma unroll
     for (int k = 0; k < PER; ++k) {
       const int c = (threadIdx.x + k * blockDim.x) * 4;
@@ -177,15 +208,18 @@ embedding_norm_kernel(const ET* __restrict__ table, const int32_t* __restrict__ 
 }  // namespace
 
 // x [T, d]; y [T, d], y_w [d], row [d], out_w [d]: 32-bit, each may be null; out [T, d] with rows out_stride apart, or null.
+// rows [., d] 32-bit, pair_row and weights [T, top], identity [T, d] bfloat16 or null: see NormStep (top 0: none of them).
 GB_EXPORT int gb_residual_norm(float* x, const float* y, const float* y_w, float y_eps, const float* row, const float* out_w,
-                               float out_eps, void* out, int out_dtype, long long out_stride, int T, int d, cudaStream_t stream) {
+                               float out_eps, void* out, int out_dtype, long long out_stride, int T, int d, const float* rows,
+                               const int32_t* pair_row, const float* weights, const void* identity, int top, cudaStream_t stream) {
   if (T <= 0) return GB_OK;
   if (d < 1 || d > 16384) return gb::fail(GB_UNSUPPORTED, "residual_norm: rows of %d (1 to 16384)", d);
   if (out != nullptr && out_stride < d) return gb::fail(GB_BAD_ARGUMENT, "residual_norm: out rows %lld apart", out_stride);
-  const NormStep p = {x, y, y_w, row, out_w, y_eps, out_eps, out_stride, d};
+  if (top < 0 || (top > 0 && (!rows || !pair_row || !weights))) return gb::fail(GB_BAD_ARGUMENT, "residual_norm: %d choices without their rows", top);
+  const NormStep p = {x, y, y_w, row, out_w, y_eps, out_eps, out_stride, d, rows, pair_row, weights, (const __nv_bfloat16*)identity, top};
   const int elem = out_dtype == GB_F32 ? 4 : 2;
   const bool vec = d % 4 == 0 && out_stride % 4 == 0 && host_aligned(x, 16) && host_aligned(y, 16) && host_aligned(y_w, 16) &&
-                   host_aligned(row, 16) && host_aligned(out_w, 16) && host_aligned(out, 4 * elem);
+                   host_aligned(row, 16) && host_aligned(out_w, 16) && host_aligned(out, 4 * elem) && host_aligned(rows, 16);
   const int quads = (d + 3) / 4;
   // few tokens: as many threads as the row has groups of four, up to two groups a thread; many: smaller blocks, more
   // of them to an SM

@@ -125,6 +125,130 @@ qk_norm_rope_append_kernel(const float* __restrict__ src, int row_stride, int q_
   }
 }
 
+// The same for heads of 16, 32, 64 or 128 channels whose rows start on 16 bytes: LANES = dim / 4 lanes hold a head in
+// registers, four neighbouring channels each, so a head is read once and its neighbours' loads are in flight together
+// (UNROLL of them a thread). Half-split pairs: the partner's channels lie rot_dims / 8 lanes away (rot_dims is a multiple
+// of eight); neighbouring pairs lie in the lane itself.
+template <typename OT>
+__device__ __forceinline__ void store4(OT* to, const float (&v)[4]);
+template <>
+__device__ __forceinline__ void store4<float>(float* to, const float (&v)[4]) { *reinterpret_cast<float4*>(to) = make_float4(v[0], v[1], v[2], v[3]); }
+template <>
+__device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16* to, const float (&v)[4]) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v[0], v[1]), hi = __floats2bfloat162_rn(v[2], v[3]);
+  *reinterpret_cast<uint2*>(to) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+}
+__device__ __forceinline__ void add4(float (&v)[4], const float* p) {
+  const float4 a = *reinterpret_cast<const float4*>(p);
+  v[0] += a.x, v[1] += a.y, v[2] += a.z, v[3] += a.w;
+}
+
+template <int LANES, typename OT>
+__global__ void __launch_bounds__(256)
+qk_norm_rope_append_wide_kernel(const float* __restrict__ src, int row_stride, int q_col, int k_col, int v_col,
+                                OT* __restrict__ q_out, OT* __restrict__ k_pool, OT* __restrict__ v_pool,
+                                const int32_t* __restrict__ positions, const int32_t* __restrict__ token_req,
+                                const int32_t* __restrict__ block_table, int table_width, int Hq, int Hkv, int vdim,
+                                const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
+                                const float* __restrict__ inv_freq, int interleaved, int rot_dims, float rot_factor, int page_size,
+                                float q_coef, int q_every, const float* __restrict__ bias, int maps) {
+  constexpr int dim = LANES * 4, UNROLL = 4;
+  __shared__ __align__(16) float sin_s[dim / 2], cos_s[dim / 2];
+  gb::pdl_launch_dependents();
+  gb::pdl_wait();
+  const int t = blockIdx.x, pos = positions[t];
+  const bool rotate = inv_freq != nullptr;
+  const float* row = src + (size_t)t * row_stride;
+  const int group = threadIdx.x / LANES, lane = threadIdx.x % LANES, groups = blockDim.x / LANES, heads = Hq + Hkv;
+  float x[UNROLL][4];
+  auto fetch = [&](int first) {
+#pragma unroll
+    for (int u = 0; u < UNROLL; ++u) {
+      const int head = first + u * groups;
+      x[u][0] = x[u][1] = x[u][2] = x[u][3] = 0.f;
+      if (head >= heads) continue;
+      add4(x[u], row + (head < Hq ? q_col + head * dim : k_col + (head - Hq) * dim) + lane * 4);
+      if (bias != nullptr) add4(x[u], bias + (size_t)head * dim + lane * 4);        // the keys' follow the queries'
+    }
+  };
+  fetch(group);
+  if (rotate)
+    for (int i = threadIdx.x; i < dim / 2; i += blockDim.x) {
+      float sn = 0.f, cs = 1.f;
+      if (i < rot_dims >> 1) {
+        sincosf((float)pos * inv_freq[i], &sn, &cs);
+        sn *= rot_factor, cs *= rot_factor;
+      }
+      sin_s[i] = sn, cos_s[i] = cs;
+    }
+  const int cached_heads = Hkv / maps;
+  long long cache_row = -1;
+  if (Hkv > 0) {
+    const int page = block_table[(size_t)token_req[t] * table_width + pos / page_size];
+    if (page >= 0) cache_row = (long long)page * cached_heads;
+  }
+  const float growth = q_every > 0 ? fmaf(q_coef, logf((float)((pos + 1) / q_every + 1)), 1.0f) : 1.0f;
+  __syncthreads();
+  const int shift = rot_dims / 8;                  // lanes between the halves of a pair
+  for (int first = group; first < (heads + groups - 1) / groups * groups; first += UNROLL * groups) {
+    if (first != group) fetch(first);
+#pragma unroll
+    for (int u = 0; u < UNROLL; ++u) {
+      const int head = first + u * groups;
+      const bool is_q = head < Hq, there = head < heads;
+      float (&v)[4] = x[u];
+      float ss = v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
+#pragma unroll
+      for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);          // (every lane of the warp is here)
+      if (is_q ? q_w != nullptr : k_w != nullptr) {
+        const float inv = 1.0f / sqrtf(ss / (float)dim + eps);
+        if (there) {
+          const float4 w = *reinterpret_cast<const float4*>((is_q ? q_w + (size_t)head * dim : k_w) + lane * 4);
+          v[0] = (v[0] * inv) * w.x, v[1] = (v[1] * inv) * w.y, v[2] = (v[2] * inv) * w.z, v[3] = (v[3] * inv) * w.w;
+        }
+      }
+      if (rotate && interleaved) {
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const float a = v[e], b = v[e + 1], cs = cos_s[lane * 2 + e / 2], sn = sin_s[lane * 2 + e / 2];
+          v[e] = a * cs - b * sn, v[e + 1] = b * cs + a * sn;
+        }
+      } else if (rotate) {
+        const bool low = lane < shift, high = lane >= shift && lane < 2 * shift;
+        const int base = (threadIdx.x & 31) - lane;
+        const int from = base + (low ? lane + shift : high ? lane - shift : lane);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float other = __shfl_sync(0xffffffffu, v[e], from);
+          if (low || high) {
+            const int i = (low ? lane : lane - shift) * 4 + e;
+            v[e] = low ? v[e] * cos_s[i] - other * sin_s[i] : v[e] * cos_s[i] + other * sin_s[i];
+          }
+        }
+      }
+      if (!there || (!is_q && cache_row < 0)) continue;
+      if (is_q) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) v[e] *= growth;
+        store4(q_out + ((size_t)t * Hq + head) * dim + lane * 4, v);
+      } else {
+        const int kh = head - Hq;
+        store4(k_pool + ((cache_row + kh / maps) * page_size + (pos % page_size)) * (maps * dim) + kh % maps * dim + lane * 4, v);
+      }
+    }
+  }
+  if (cache_row >= 0) {
+    const float* vs = row + v_col;
+    const float* bs = bias ? bias + (size_t)heads * dim : nullptr;
+    for (int e = threadIdx.x * 4; e < cached_heads * vdim; e += blockDim.x * 4) {
+      float v[4] = {0.f, 0.f, 0.f, 0.f};
+      add4(v, vs + e);
+      if (bs != nullptr) add4(v, bs + e);
+      store4(v_pool + ((cache_row + e / vdim) * page_size + (pos % page_size)) * vdim + e % vdim, v);
+    }
+  }
+}
+
 enum { ACT_SIGMOID = 0, ACT_SILU = 1, ACT_RELU2 = 2, ACT_TANH = 3, ACT_GELU = 4 };
 
 __device__ __forceinline__ float act(float z, int kind) {
@@ -328,6 +452,22 @@ GB_EXPORT int gb_qk_norm_rope_append(const float* src, int row_stride, int q_col
   if (Hkv > 0 && (!k_pool || !v_pool || !block_table || page_size < 1))
     return gb::fail(GB_BAD_ARGUMENT, "qk_norm_rope_append: kv heads given without a cache to store them in");
   const int heads = Hq + Hkv;
+  const int elem = out_dtype == GB_F32 ? 4 : 2;
+  const auto on = [](const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; };
+  const bool wide = (dim == 16 || dim == 32 || dim == 64 || dim == 128) && (inv_freq == nullptr || interleaved || rot_dims % 8 == 0) &&
+                    ((row_stride | q_col | k_col | v_col | (Hkv > 0 ? vdim : 0)) & 3) == 0 && on(src, 16) && on(q_w, 16) && on(k_w, 16) && on(bias, 16) &&
+                    on(q_out, 4 * elem) && on(k_pool, 4 * elem) && on(v_pool, 4 * elem);
+  if (wide)
+    return GB_DISPATCH_DTYPE(out_dtype, OT, [&]() -> int {
+      auto kernel = dim == 16 ? qk_norm_rope_append_wide_kernel<4, OT> : dim == 32 ? qk_norm_rope_append_wide_kernel<8, OT>
+                    : dim == 64 ? qk_norm_rope_append_wide_kernel<16, OT> : qk_norm_rope_append_wide_kernel<32, OT>;
+      const int needed = (heads * (dim / 4) + 3) / 4;          // threads for four heads a group
+      return gb::check_pdl_launch(
+          gb::launch_pdl(kernel, dim3(T), dim3(needed > 128 ? 256 : needed > 64 ? 128 : 64), 0, stream, dim3(1, 1, 1), src, row_stride,
+                         q_col, k_col, v_col, (OT*)q_out, (OT*)k_pool, (OT*)v_pool, positions, token_req, block_table, table_width, Hq,
+                         Hkv, vdim, q_w, k_w, eps, inv_freq, interleaved, rot_dims, rot_factor, page_size, q_coef, q_every, bias, maps),
+          "qk_norm_rope_append");
+    });
   const int block = heads >= 8 ? 256 : (heads >= 4 ? 128 : 64);
   return GB_DISPATCH_DTYPE(out_dtype, OT, [&]() -> int {
     return gb::check_pdl_launch(

@@ -74,6 +74,15 @@ class PendingNorm:
         return self.norm.forward(ctx, self.x)
 
 
+class ExpertRows:
+    """What routed experts leave for the pass that reads their sum: ``rows [., d]`` (32-bit), a row per (token, choice) pair;
+    ``pair_row``: device address of the int32 list of the pairs' rows (-1: none); ``weights [T, top]``; ``identity`` (bfloat16 ``[T, d]`` or None):
+    what a pair without a row stands for; ``base`` (32-bit ``[T, d]`` or None) is added."""
+
+    def __init__(self, rows, pair_row, weights, identity, base):
+        self.rows, self.pair_row, self.weights, self.identity, self.base = rows, pair_row, weights, identity, base
+
+
 class CudaOps:
     """Hand-written sm_100a kernels. ``tensor_cores=False`` keeps every matrix
     product and the attention on the plain 32-bit-arithmetic kernels (the true
@@ -231,7 +240,7 @@ class CudaOps:
 
     _MEMORY_SIGNATURES = {
         "gb_residual_norm": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_float, c_void_p, c_int, c_longlong, c_int, c_int,
-                             c_void_p],
+                             c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
         "gb_embedding_norm": [c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
         "gb_memory_gates": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p,
                             c_void_p, c_int, c_int, c_void_p],
@@ -308,7 +317,7 @@ class CudaOps:
                                  c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
             "gb_head_gemm": [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_longlong, c_int, c_int, c_void_p, c_int,
                              c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
-            "gb_route_topk": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
+            "gb_route_topk": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
                               c_int, c_void_p, c_void_p, c_void_p],
             "gb_moe_gate_up": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                c_int, c_float, c_void_p, c_void_p],
@@ -749,6 +758,9 @@ class CudaOps:
         self.gated_act(tmp, act, kind, limit, group)
 
     # ------------------------------------------------------------------ routed experts
+    #: tokens from which the router's logits are a product of their own
+    ROUTER_PRODUCT_TOKENS = 256
+
     ROUTER_SCORES = {"softmax_chosen": 0, "sigmoid": 1, "softmax_all": 2}
 
     def route_topk(self, h, w_router, bias, top, ids, weights, score: str = "softmax_chosen", correction=None, groups=None):
@@ -769,8 +781,13 @@ class CudaOps:
         _need(ids.dtype == torch.int32 and weights.dtype == torch.float32 and ids.shape == (T, top)
               and weights.shape == (T, top) and ids.is_contiguous() and weights.is_contiguous(), "route_topk: outputs")
         _need(bias is None or (bias.dtype == torch.float32 and bias.numel() == E), "route_topk: a float32 bias")
+        logits = None
+        if self.tc is not None and h.dtype == w_router.dtype == torch.bfloat16 and T >= self.ROUTER_PRODUCT_TOKENS and K % 8 == 0:
+            # many tokens: the logits as one product on the tensor cores (32-bit sums)
+            logits = self.private_ws.get("router_logits", (T, E), torch.float32)
+            self.linear(h, w_router, logits)
         self._check(self.mixers, self.mixers.gb_route_topk(
-            h.data_ptr(), _tag(h, "router input"), w_router.data_ptr(), _ptr(bias), _tag(w_router, "router"),
+            h.data_ptr(), _tag(h, "router input"), w_router.data_ptr(), _ptr(logits), _ptr(bias), _tag(w_router, "router"),
             T, E, K, int(top), self.ROUTER_SCORES[score], _ptr(correction), int(count), int(keep), ids.data_ptr(), weights.data_ptr(),
             self._stream()), "route_topk")
 
@@ -814,7 +831,7 @@ class CudaOps:
               and w_up.shape[2] == K and act.shape == (T, top, F), "moe_up: shapes")
         self._check(self.mixers, self.mixers.gb_moe_up(
             h.data_ptr(), _tag(h, "h"), w_up.data_ptr(), _tag(w_up, "w"), ids.data_ptr(), act.data_ptr(), _tag(act, "act"), T, top,
-            F, K, self.UNARY_ACTS[kind], _ptr(in_scale), self._stream()), "moe_up")
+            E, F, K, self.UNARY_ACTS[kind], _ptr(in_scale), self._stream()), "moe_up")
 
     def pack_expert_gate_up(self, gates, ups):
         """The experts' gate and up matrices stacked, in the layout ``routed_feed_forward`` wants:
@@ -830,12 +847,27 @@ class CudaOps:
     #: the experts' last pass may also compute a norm without statistics of the residual it writes (``then``)
     fuses_tanh_norms = True
 
+    #: the experts' rows may be left for the pass that reads their sum (``expert_rows``)
+    leaves_expert_rows = True
+
+    def expert_rows(self, ctx, h, w_gate_up, w_down, ids, weights, kind: str, limit: float, identity: bool = False, base=None):
+        """``routed_feed_forward`` of gated experts without its last step: an ``ExpertRows`` whose sum, with ``base`` (32-bit ``[T,
+        N]`` or None), is the feed-forward's output, for ``residual_norm`` to add up as it reads it; None where the sizes run
+        on the plain kernels."""
+        if getattr(w_gate_up, "gb_group", 0) != 64 or self.tc is None or h.dtype != torch.bfloat16:
+            return None
+        left = []
+        x = torch.empty((ids.shape[0], 0), device=h.device)          # only its rows count: nothing is added to it
+        self.routed_feed_forward(ctx, h, w_gate_up, w_down, ids, weights, x, kind, limit, identity=identity, left=left)
+        rows, pair_row = left
+        return ExpertRows(rows, pair_row, weights, h if identity else None, base)
+
     #: (token, choice) pairs from which the routed experts run on the tcgen05 grouped product
     GROUPED_TC_PAIRS = 1024
 
     def routed_feed_forward(self, ctx, h, w_gate_up, w_down, ids, weights, x, kind: str, limit: float,
                             alpha: float = 1.0, scale_input: bool = False, gated: bool = True, then=None,
-                            identity: bool = False):
+                            identity: bool = False, left: Optional[list] = None):
         """``x[t] += alpha * sum_j weights[t, j] * expert_{ids[t, j]}(h[t])`` with the experts'
         weights stacked: ``w_gate_up`` from ``pack_expert_gate_up``, ``w_down [E, N, F]``. Without ``gated``:
         ``w_gate_up`` is ``[E, F, K]``, the up rows alone, and ``kind`` an activation of one value.
@@ -844,7 +876,8 @@ class CudaOps:
         whether it did.
         ``scale_input``: the weight multiplies what goes into the expert instead,
         ``sum_j expert(weights[t, j] * h[t])``. An id beyond the ``E`` experts stands for no expert: its term is
-        ``weights[t, j] * h[t]`` with ``identity``, else nothing."""
+        ``weights[t, j] * h[t]`` with ``identity``, else nothing. ``left`` (tensor-core sizes): nothing is added to ``x``; the list gets
+        the pairs' rows and the row of every pair."""
         _need(not identity or (h.shape[1] == w_down.shape[1] and not scale_input), "routed_feed_forward: an expert that returns its input")
         T, top = ids.shape
         E, N, F = w_down.shape
@@ -852,7 +885,7 @@ class CudaOps:
         packed = getattr(w_gate_up, "gb_group", 0) == 64
         grouped = packed if gated else (self.tc is not None and h.dtype == torch.bfloat16 and K % 8 == 0 and F % 8 == 0 and E <= 4096)
         if grouped and T * top >= self.GROUPED_TC_PAIRS and self._routed_tcgen05(ctx, h, w_gate_up, w_down, ids, weights,
-                                                                                x, kind, limit, alpha, scale_input, gated, then, identity):
+                                                                                x, kind, limit, alpha, scale_input, gated, then, identity, left):
             return then is not None
         norm = self._then_norm(then, T, N)
         if grouped:
@@ -860,7 +893,8 @@ class CudaOps:
             self._on_device(h, w_gate_up, w_down, ids, weights, x)
             _need(h.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous() and ids.is_contiguous()
                   and weights.is_contiguous() and x.is_contiguous() and x.dtype == torch.float32
-                  and tuple(w_gate_up.shape) == (E, 128 * ((F + 63) // 64) if gated else F, K) and x.shape == (T, N) and ids.dtype == torch.int32
+                  and tuple(w_gate_up.shape) == (E, 128 * ((F + 63) // 64) if gated else F, K) and (left is not None or x.shape == (T, N))
+                  and ids.dtype == torch.int32
                   and weights.dtype == torch.float32 and w_gate_up.dtype == w_down.dtype == torch.bfloat16,
                   "routed_feed_forward: shapes")
             L = self.mixers
@@ -869,10 +903,12 @@ class CudaOps:
             act = ctx.ws.get("expert_act", (T * top, F), torch.bfloat16)
             y = ctx.ws.get("expert_rows", (T * top, N), torch.float32)
             self._check(L, L.gb_moe_grouped(
-                h.data_ptr(), w_gate_up.data_ptr(), w_down.data_ptr(), ids.data_ptr(), weights.data_ptr(), x.data_ptr(),
-                T, top, E, F, K, N, self.GATE_ACTS[kind] if gated else self.UNARY_ACTS[kind], float(limit), float(alpha),
+                h.data_ptr(), w_gate_up.data_ptr(), w_down.data_ptr(), ids.data_ptr(), weights.data_ptr(),
+                None if left is not None else x.data_ptr(), T, top, E, F, K, N, self.GATE_ACTS[kind] if gated else self.UNARY_ACTS[kind], float(limit), float(alpha),
                 1 if gated else 2, int(scale_input), index.data_ptr(),
-                act.data_ptr(), y.data_ptr(), *norm, int(identity), self._stream()), "moe_grouped", 4)
+                act.data_ptr(), y.data_ptr(), *norm, int(identity), self._stream()), "moe_grouped", 4 if left is None else 3)
+            if left is not None:
+                left += [y, index.data_ptr() + 4 * T * top]
             return then is not None
         act = ctx.ws.get("expert_act", (T, top, F), h.dtype)
         if gated:
@@ -892,7 +928,7 @@ class CudaOps:
         return (out.data_ptr(), w.data_ptr(), b.data_ptr(), float(alpha))
 
     def _routed_tcgen05(self, ctx, h, w_gate_up, w_down, ids, weights, x, kind, limit, alpha, scale_input=False,
-                        gated=True, then=None, identity=False) -> bool:
+                        gated=True, then=None, identity=False, left=None) -> bool:
         """Many pairs: sorted by expert into blocks of 128 rows (padding rows zero), then the two
         products on the tcgen05 many-token kernel with each block's expert read from a list."""
         T, top = ids.shape
@@ -911,7 +947,7 @@ class CudaOps:
             return False
         self._on_device(h, w_gate_up, w_down, ids, weights, x)
         _need(h.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous() and ids.is_contiguous()
-              and weights.is_contiguous() and x.is_contiguous() and x.dtype == torch.float32 and x.shape == (T, N)
+              and weights.is_contiguous() and x.is_contiguous() and x.dtype == torch.float32 and (left is not None or x.shape == (T, N))
               and ids.dtype == torch.int32 and weights.dtype == torch.float32
               and h.dtype == w_gate_up.dtype == w_down.dtype == torch.bfloat16, "routed_feed_forward: shapes")
         index = ctx.ws.get("expert_index_padded", (T * top + 2 * blocks,), torch.int32)
@@ -926,6 +962,9 @@ class CudaOps:
         else:
             tc.grouped(a, w_gate_up, act, F, E, block_gu, 0, gate_act=tc.STORE_ACTS[kind])
         tc.grouped(act, w_down, y, N, E, block_dn, 0)
+        if left is not None:
+            left += [y, index.data_ptr()]
+            return True
         self._check(L, L.gb_moe_combine(y.data_ptr(), index.data_ptr(), None if scale_input else weights.data_ptr(), x.data_ptr(), T, top, N,
                                         float(alpha), *self._then_norm(then, T, N), h.data_ptr() if identity else None, self._stream()),
                     "moe_combine")
@@ -1493,7 +1532,12 @@ class CudaOps:
     def residual_norm(self, x, y=None, weight=None, eps: float = 0.0, row=None, then_weight=None, then_eps: float = 0.0, out=None):
         """``x += rms(y) * weight`` (``weight`` None: ``x += y``) and ``x += row`` on the 32-bit residual ``x [T, d]``, ``y`` 32-bit
         ``[T, d]`` or None, ``row [d]`` or None; then ``out = rms(x) * then_weight`` (``then_weight`` None: ``out = x``) in
-        ``out``'s dtype (a column range of a wider row will do). Vectors are 32-bit. One pass."""
+        ``out``'s dtype (a column range of a wider row will do). Vectors are 32-bit. ``y`` may be an ``ExpertRows``. One pass."""
+        experts, y = (y, y.base) if isinstance(y, ExpertRows) else (None, y)
+        gather = (None, None, None, None, 0)
+        if experts is not None:
+            _need(experts.rows.shape[1] == x.shape[1] and tuple(experts.weights.shape[:1]) == tuple(x.shape[:1]), "residual_norm: the experts' rows")
+            gather = (experts.rows.data_ptr(), experts.pair_row, experts.weights.data_ptr(), _ptr(experts.identity), experts.weights.shape[1])
         self._on_device(x, y, weight, row, then_weight, out)
         _need(x.dtype == torch.float32 and x.is_contiguous() and x.dim() == 2, "residual_norm: x must be float32 [T, d]")
         T, d = x.shape
@@ -1504,7 +1548,7 @@ class CudaOps:
         L = self.memory_lib
         self._check(L, L.gb_residual_norm(
             x.data_ptr(), _ptr(y), _ptr(weight), float(eps), _ptr(row), _ptr(then_weight), float(then_eps), _ptr(out),
-            _tag(out, "residual_norm out") if out is not None else GB_F32, out.stride(0) if out is not None else d, T, d, self._stream()),
+            _tag(out, "residual_norm out") if out is not None else GB_F32, out.stride(0) if out is not None else d, T, d, *gather, self._stream()),
             "residual_norm")
 
     def embedding_norm(self, table, ids, weight, eps, x, pair=None):

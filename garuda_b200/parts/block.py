@@ -527,4 +527,5 @@ class SandwichNormBlock:
                         NormedInput(self.feed_forward_norm) if ff is not None else last, 0 if ff is not None else 1)
         if ff is None:
             return h2
-        return self._join(ctx, x, ff.forward(ctx, h2), self.feed_forward_post_norm, last, 1)
+        kw = {"leave_rows": True} if getattr(ff, "leaves_rows", False) else {}
+        return self._join(ctx, x, ff.forward(ctx, h2, **kw), self.feed_forward_post_norm, last, 1)

@@ -114,20 +114,35 @@ class RoutedExperts(FeedForward):
         """Whether ``forward`` takes ``emit_norm``, a ``DynamicTanh`` of the residual that this part is the last to write."""
         return not self.shared_inner
 
-    def forward(self, ctx, h, residual=None, alpha: float = 1.0, emit_norm=None):
+    #: ``forward`` takes ``leave_rows``: the output may be left as rows that the pass behind adds up
+    leaves_rows = True
+
+    def forward(self, ctx, h, residual=None, alpha: float = 1.0, emit_norm=None, leave_rows: bool = False):
         ops, ws = self.ops, ctx.ws
         T = h.shape[0]
         target = residual
         shared_first = target is None and self.shared_inner
+        leave_rows = leave_rows and self.gated and not self.scale_input and getattr(ops, "leaves_expert_rows", False)
         if target is None:
             target = ws.get("ffn_out", (T, self.width), torch.float32)
             alpha = 1.0
             if shared_first:
                 self._shared(ctx, h, target, accumulate=False)       # stored: the routed ones are added to it
-            else:
+            elif not leave_rows:
                 target.zero_()
         ids = ws.get("expert_ids", (T, self.top), torch.int32)
         weights = ws.get("expert_weights", (T, self.top), torch.float32)
+        if leave_rows and residual is None:
+            ops.route_topk(h, self.w_router, self.b_router, self.top, ids, weights, score=self.router_score, **self.choice)
+            rows = ops.expert_rows(ctx, h, self.w_gate_up, self.w_down, ids, weights, self.activation, self.limit,
+                                   identity=bool(self.identity), base=target if shared_first else None)
+            if rows is not None:
+                return rows
+            if not shared_first:
+                target.zero_()
+            ops.routed_feed_forward(ctx, h, self.w_gate_up, self.w_down, ids, weights, target, self.activation, self.limit,
+                                    identity=bool(self.identity))
+            return target
         if self.router_score == "softmax_chosen" and not self.scale_input and self.gated and not self.choice and not self.identity:
             ops.route_topk(h, self.w_router, self.b_router, self.top, ids, weights)
             ops.routed_feed_forward(ctx, h, self.w_gate_up, self.w_down, ids, weights, target, self.activation,

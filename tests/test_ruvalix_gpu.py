@@ -105,21 +105,49 @@ def test_experts_that_return_their_input(both, T, E, identity, K, F, top, shared
         close(got, want, dt, f"experts, identity {on}")
 
 
-@pytest.mark.parametrize("H,G,dim,vdim", [(4, 2, 24, 40), (3, 1, 15, 9), (8, 8, 64, 32), (2, 1, 128, 16)])
-@pytest.mark.parametrize("turned,factor,layout", [(8, 1.3, "half"), (14, 1.0, "half"), (0, 1.0, "half"), (6, 0.9, "interleaved")])
+@pytest.mark.parametrize("T", [1, 9, 150, 700])
+def test_experts_rows_are_added_up_by_the_pass_behind_them(T):
+    """Few pairs and many, with and without a base and experts that return their input: the pass over the residual behind
+    them gives what it gives behind their sum; sizes of the plain kernels leave no rows."""
+    from garuda_b200.kernels.ops import CudaOps
+    ops, bf = CudaOps("cuda:0"), torch.bfloat16
+    for E, identity, K, F, top, leaves in ((6, 3, 128, 64, 3, True), (5, 0, 1032, 40, 2, True), (6, 3, 44, 24, 3, False)):
+        h, down = rnd(T, K, dtype=bf, seed=1).cuda(), rnd(E, K, F, dtype=bf, scale=0.3, seed=2).cuda()
+        gu = ops.pack_expert_gate_up([rnd(F, K, dtype=bf, scale=0.2, seed=9 + e).cuda() for e in range(E)], [rnd(F, K, dtype=bf, scale=0.2, seed=40 + e).cuda() for e in range(E)])
+        ids = torch.stack([torch.randperm(E + identity)[:top] for _ in range(T)]).to(torch.int32).cuda()
+        wts, base, x = torch.rand(T, top).cuda(), rnd(T, K, seed=3).cuda(), rnd(T, K, seed=4).cuda()
+        w, w2 = rnd(K, seed=5).cuda(), rnd(K, seed=6).cuda()
+        for b in (base, None):
+            rows = ops.expert_rows(_Ctx(), h, gu, down, ids, wts, "silu", 0.0, identity=identity > 0, base=b)
+            assert (rows is not None) == leaves
+            if not leaves:
+                continue
+            y = b.clone() if b is not None else torch.zeros(T, K, device="cuda")
+            ops.routed_feed_forward(_Ctx(), h, gu, down, ids, wts, y, "silu", 0.0, identity=identity > 0)
+            x1, x2, o1, o2 = x.clone(), x.clone(), torch.empty(T, K, dtype=bf, device="cuda"), torch.empty(T, K, dtype=bf, device="cuda")
+            ops.residual_norm(x1, y, w, 1e-5, then_weight=w2, then_eps=1e-5, out=o1)
+            ops.residual_norm(x2, rows, w, 1e-5, then_weight=w2, then_eps=1e-5, out=o2)
+            close(x2, x1.cpu(), torch.float32, "residual", 1e-5)
+            close(o2, o1.cpu(), bf, "normed", 1e-2)
+
+
+@pytest.mark.parametrize("H,G,dim,vdim", [(4, 2, 24, 40), (3, 1, 15, 9), (8, 8, 64, 32), (2, 1, 128, 16), (6, 2, 16, 12), (5, 5, 32, 8)])
+@pytest.mark.parametrize("turned,factor,layout", [(8, 1.3, "half"), (14, 1.0, "half"), (0, 1.0, "half"), (6, 0.9, "interleaved"), (16, 1.1, "half")])
 def test_biased_normed_maps_into_pages(both, H, G, dim, vdim, turned, factor, layout):
     """A bias, the norm, a rotation of the first channels at positions across pages, two maps to a cached row."""
     from garuda_b200.parts.rotary import RotaryParams
     ops, ref, dt = both
-    ps = 8
+    if turned > dim:
+        pytest.skip("not that many channels")
+    ps, lead = 8, 4 if dim % 16 == 0 else 1           # (rows that start on 16 bytes and rows that do not)
     b, table, pages = step_batch([5, 1, 60, 2], [0, 62, 3, 5], [2, 0, 3, 1], ps)
     bg = batches(b)[0].batch
     rot = RotaryParams(100.0, turned, layout == "interleaved", tuple(1.0 / (i + 1.5) for i in range(turned // 2)), factor) if turned else None
     T, cols = b.num_tokens, 2 * (H + G) * dim + G * vdim
-    row, bias, qw, kw = rnd(T, cols + 3, seed=1), rnd(cols, seed=2), rnd(2 * H, dim, seed=3), rnd(dim, seed=4)
+    row, bias, qw, kw = rnd(T, cols + lead + 4 - (cols + lead) % 4, seed=1), rnd(cols, seed=2), rnd(2 * H, dim, seed=3), rnd(dim, seed=4)
     kp, vp, q = torch.zeros(pages, G, ps, 2 * dim, dtype=dt), torch.zeros(pages, G, ps, vdim, dtype=dt), torch.zeros(T, 2 * H, dim, dtype=dt)
     kg, vg, qg = kp.cuda(), vp.cuda(), q.cuda()
-    c = (1, 1 + 2 * H * dim, 1 + 2 * (H + G) * dim)
+    c = (lead, lead + 2 * H * dim, lead + 2 * (H + G) * dim)
     ref.qk_norm_rope_append(row, c, q, kp, vp, b.positions, b.token_req, table, 2 * H, 2 * G, dim, vdim, qw, kw, 1e-5, rot, ps, bias=bias, maps=2)
     ops.qk_norm_rope_append(row.cuda(), c, qg, kg, vg, bg.positions, bg.token_req, table.cuda(), 2 * H, 2 * G, dim, vdim, qw.cuda(), kw.cuda(), 1e-5,
                             rot, ps, bias=bias.cuda(), maps=2)
@@ -263,7 +291,7 @@ def test_chunks_on_the_tensor_cores_keep_32_bit_memories(H, D, P):
 def check(got, ref, dtype, what, name):
     """Per position, the largest difference as a fraction of the largest logit. 32-bit: every position
     within 2e-4 (sums in another order than the 64-bit plain model's). bfloat16: nine positions in ten
-    within 0.06 and the median within 0.015, the rest finite: with sharpened random weights a router's
+    within 0.06 and the median of sixteen and more within 0.015, the rest finite: with sharpened random weights a router's
     close call, a sharp softmax or two maps that nearly cancel turn the rounding of an input into a large change at a
     few positions, in the plain model itself; a fault of a kernel, a mask or a state shows at most positions."""
     scale = float(np.abs(ref).max())
@@ -275,7 +303,7 @@ def check(got, ref, dtype, what, name):
         return
     over = int((err > 0.06).sum())
     assert over <= max(1, len(err) // 10), f"{what}: {over} of {len(err)} positions beyond 0.06 (largest {err.max():.3e})"
-    assert np.median(err) <= 0.015, f"{what}: median {np.median(err):.3e}"
+    assert len(err) < 16 or np.median(err) <= 0.015, f"{what}: median {np.median(err):.3e}"
 
 
 @pytest.fixture(scope="module", params=[(n, d) for n in CASES for d in ("float32", "bfloat16")], ids=lambda p: f"{p[0]}-{p[1]}")
