@@ -21,7 +21,7 @@ constexpr int MAX_TOP = 32;
 // without it. groups > 0: the experts form so many equal groups of neighbours, a group's score is its best
 // expert's, and only experts of the `keep` best groups (the lower index first among equals) can be chosen.
 template <typename HT, typename WT>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(1024)
 route_topk_kernel(const HT* __restrict__ h, const WT* __restrict__ w, const float* __restrict__ logits,
                   const float* __restrict__ bias, int T, int E, int K, int top, int mode, const float* __restrict__ correction, int groups, int keep,
                   int32_t* __restrict__ ids, float* __restrict__ weights) {
@@ -45,7 +45,7 @@ route_topk_kernel(const HT* __restrict__ h, const WT* __restrict__ w, const floa
     const WT* wr = w + (size_t)e * K;
     float acc = 0.f;
     if (sizeof(WT) == 2 && K % 8 == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0) {        // eight neighbouring weights in one load (rows start on 16 bytes)
-#pragma unroll 4
+#pragma unroll 8
       for (int k = lane * 8; k < K; k += 256) {
         const uint4 v = *reinterpret_cast<const uint4*>(wr + k);
         const uint32_t pairs[4] = {v.x, v.y, v.z, v.w};
@@ -261,6 +261,8 @@ GB_EXPORT int gb_route_topk(const void* h, int h_dtype, const void* w, const flo
     return gb::fail(GB_BAD_ARGUMENT, "route_topk: %d of %d groups of %d experts, %d chosen", keep, groups, E, top);
   const size_t smem = (size_t)(3 * E + (logits != nullptr ? 0 : K)) * sizeof(float);
   if (smem > 200 * 1024) return gb::fail(GB_UNSUPPORTED, "route_topk: width %d", K);
+  // few tokens: a warp for every expert, up to a block's 32
+  const int threads = logits != nullptr ? 32 : (T < 148 && E > 8 ? (E < 32 ? E * 32 : 1024) : 256);
   return GB_DISPATCH_DTYPE(h_dtype, HT, [&]() -> int {
     return GB_DISPATCH_DTYPE(w_dtype, WT, [&]() -> int {
       if (smem > 48 * 1024) {     // rare (rows beyond 12,000 values): asked for at every such launch
@@ -268,7 +270,7 @@ GB_EXPORT int gb_route_topk(const void* h, int h_dtype, const void* w, const flo
         if (e != cudaSuccess) return gb::fail(GB_CUDA_ERROR, "route_topk: %s", cudaGetErrorString(e));
       }
       return gb::check_pdl_launch(
-          gb::launch_pdl(route_topk_kernel<HT, WT>, dim3(T), dim3(logits != nullptr ? 32 : 256), smem, stream,
+          gb::launch_pdl(route_topk_kernel<HT, WT>, dim3(T), dim3(threads), smem, stream,
                          dim3(1, 1, 1), (const HT*)h, (const WT*)w, logits, bias, T, E, K, top, mode, correction, groups, keep, ids, weights),
           "route_topk");
     });

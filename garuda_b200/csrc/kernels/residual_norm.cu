@@ -46,11 +46,11 @@ struct NormStep {
   int d;
   // routed experts' rows, added to y: sum_j weights[t][j] * rows[pair_row[t top + j]], j in the router's order; a pair without a row
   // stands for identity[t] (null: nothing). top 0: none.
-  const float* rows;         // [., d]
+  const float* rows;         // [num_rows, d]
   const int32_t* pair_row;
   const float* weights;      // [T, top]
   const __nv_bfloat16* identity;
-  int top;
+  int top, num_rows;
 };
 
 // One block per token; a thread keeps PER groups of four neighbouring channels of the row in registers from the
@@ -100,7 +100,7 @@ residual_norm_kernel(const NormStep p, OT* __restrict__ out) {
         const int c = (threadIdx.x + k * blockDim.x) * 4;
         if (c >= d) continue;
         float v[4] = {0.f, 0.f, 0.f, 0.f};
-        if (from >= 0) {
+        if (from >= 0 && from < p.num_rows) {
           load4(p.rows + (size_t)from * d, c, v);
         } else if (p.identity != nullptr) {
 #pragma unroll
@@ -208,15 +208,16 @@ embedding_norm_kernel(const ET* __restrict__ table, const int32_t* __restrict__ 
 }  // namespace
 
 // x [T, d]; y [T, d], y_w [d], row [d], out_w [d]: 32-bit, each may be null; out [T, d] with rows out_stride apart, or null.
-// rows [., d] 32-bit, pair_row and weights [T, top], identity [T, d] bfloat16 or null: see NormStep (top 0: none of them).
+// rows [num_rows, d] 32-bit, pair_row and weights [T, top], identity [T, d] bfloat16 or null: see NormStep (top 0: none of them).
 GB_EXPORT int gb_residual_norm(float* x, const float* y, const float* y_w, float y_eps, const float* row, const float* out_w,
                                float out_eps, void* out, int out_dtype, long long out_stride, int T, int d, const float* rows,
-                               const int32_t* pair_row, const float* weights, const void* identity, int top, cudaStream_t stream) {
+                               const int32_t* pair_row, const float* weights, const void* identity, int top, int num_rows,
+                               cudaStream_t stream) {
   if (T <= 0) return GB_OK;
   if (d < 1 || d > 16384) return gb::fail(GB_UNSUPPORTED, "residual_norm: rows of %d (1 to 16384)", d);
   if (out != nullptr && out_stride < d) return gb::fail(GB_BAD_ARGUMENT, "residual_norm: out rows %lld apart", out_stride);
   if (top < 0 || (top > 0 && (!rows || !pair_row || !weights))) return gb::fail(GB_BAD_ARGUMENT, "residual_norm: %d choices without their rows", top);
-  const NormStep p = {x, y, y_w, row, out_w, y_eps, out_eps, out_stride, d, rows, pair_row, weights, (const __nv_bfloat16*)identity, top};
+  const NormStep p = {x, y, y_w, row, out_w, y_eps, out_eps, out_stride, d, rows, pair_row, weights, (const __nv_bfloat16*)identity, top, num_rows};
   const int elem = out_dtype == GB_F32 ? 4 : 2;
   const bool vec = d % 4 == 0 && out_stride % 4 == 0 && host_aligned(x, 16) && host_aligned(y, 16) && host_aligned(y_w, 16) &&
                    host_aligned(row, 16) && host_aligned(out_w, 16) && host_aligned(out, 4 * elem) && host_aligned(rows, 16);

@@ -76,7 +76,7 @@ class PendingNorm:
 
 class ExpertRows:
     """What routed experts leave for the pass that reads their sum: ``rows [., d]`` (32-bit), a row per (token, choice) pair;
-    ``pair_row``: device address of the int32 list of the pairs' rows (-1: none); ``weights [T, top]``; ``identity`` (bfloat16 ``[T, d]`` or None):
+    ``pair_row [T * top]`` (int32): every pair's row (-1: none); ``weights [T, top]``; ``identity`` (bfloat16 ``[T, d]`` or None):
     what a pair without a row stands for; ``base`` (32-bit ``[T, d]`` or None) is added."""
 
     def __init__(self, rows, pair_row, weights, identity, base):
@@ -240,7 +240,7 @@ class CudaOps:
 
     _MEMORY_SIGNATURES = {
         "gb_residual_norm": [c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_float, c_void_p, c_int, c_longlong, c_int, c_int,
-                             c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
+                             c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "gb_embedding_norm": [c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
         "gb_memory_gates": [c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p,
                             c_void_p, c_int, c_int, c_void_p],
@@ -908,7 +908,7 @@ class CudaOps:
                 1 if gated else 2, int(scale_input), index.data_ptr(),
                 act.data_ptr(), y.data_ptr(), *norm, int(identity), self._stream()), "moe_grouped", 4 if left is None else 3)
             if left is not None:
-                left += [y, index.data_ptr() + 4 * T * top]
+                left += [y, index[T * top:2 * T * top]]
             return then is not None
         act = ctx.ws.get("expert_act", (T, top, F), h.dtype)
         if gated:
@@ -963,7 +963,7 @@ class CudaOps:
             tc.grouped(a, w_gate_up, act, F, E, block_gu, 0, gate_act=tc.STORE_ACTS[kind])
         tc.grouped(act, w_down, y, N, E, block_dn, 0)
         if left is not None:
-            left += [y, index.data_ptr()]
+            left += [y, index[:T * top]]
             return True
         self._check(L, L.gb_moe_combine(y.data_ptr(), index.data_ptr(), None if scale_input else weights.data_ptr(), x.data_ptr(), T, top, N,
                                         float(alpha), *self._then_norm(then, T, N), h.data_ptr() if identity else None, self._stream()),
@@ -1534,10 +1534,16 @@ class CudaOps:
         ``[T, d]`` or None, ``row [d]`` or None; then ``out = rms(x) * then_weight`` (``then_weight`` None: ``out = x``) in
         ``out``'s dtype (a column range of a wider row will do). Vectors are 32-bit. ``y`` may be an ``ExpertRows``. One pass."""
         experts, y = (y, y.base) if isinstance(y, ExpertRows) else (None, y)
-        gather = (None, None, None, None, 0)
+        gather = (None, None, None, None, 0, 0)
         if experts is not None:
-            _need(experts.rows.shape[1] == x.shape[1] and tuple(experts.weights.shape[:1]) == tuple(x.shape[:1]), "residual_norm: the experts' rows")
-            gather = (experts.rows.data_ptr(), experts.pair_row, experts.weights.data_ptr(), _ptr(experts.identity), experts.weights.shape[1])
+            top = experts.weights.shape[1]
+            self._on_device(experts.rows, experts.pair_row, experts.weights, experts.identity)
+            _need(experts.rows.shape[1] == x.shape[1] and experts.weights.shape[0] == x.shape[0] and experts.weights.is_contiguous()
+                  and experts.pair_row.dtype == torch.int32 and experts.pair_row.numel() == x.shape[0] * top
+                  and (experts.identity is None or (experts.identity.shape == x.shape and experts.identity.is_contiguous()
+                                                    and experts.identity.dtype == torch.bfloat16)), "residual_norm: the experts' rows")
+            gather = (experts.rows.data_ptr(), experts.pair_row.data_ptr(), experts.weights.data_ptr(), _ptr(experts.identity), top,
+                      experts.rows.shape[0])
         self._on_device(x, y, weight, row, then_weight, out)
         _need(x.dtype == torch.float32 and x.is_contiguous() and x.dim() == 2, "residual_norm: x must be float32 [T, d]")
         T, d = x.shape
